@@ -8,7 +8,8 @@
 // blocks share an SM; rows padded by 16 bytes so that ldmatrix is free of bank conflicts at every row length). A warp owns 16 query rows and a slice of the
 // value columns; with two slices (DV above 256) both warps of a row compute the same scores. Scores, softmax and the
 // weighted sums are float32; the softmax weights meet the values as two bfloat16 terms (the weight rounded, and what
-// the rounding left over), so that no weight is rounded to 8 bits. A sink joins the denominator at the end. The keys
+// the rounding left over), so that no weight is rounded to 8 bits. A sink joins the denominator at the end, a gate per token and head multiplies the
+// result. With a window a block starts at the tile of the first key that any of its rows sees. The keys
 // of a row can be cut into splits (grid.y) whose partial sums a second kernel merges: that is how a step of few
 // decoded tokens fills the GPU.
 //
@@ -54,7 +55,8 @@ attention_latent_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
                         const int* __restrict__ block_table, int max_blocks, __nv_bfloat16* __restrict__ out,
                         int out_stride, float* __restrict__ part_o, float* __restrict__ part_ml, int H, int DK, int DV,
                         int P, int n_pages, float scale_log2e, int n_splits, int* __restrict__ error_flag,
-                        const float* __restrict__ sink, int n_bufs) {
+                        const float* __restrict__ sink, int n_bufs, int window, const __nv_bfloat16* __restrict__ gate,
+                        int gate_stride) {
     extern __shared__ __align__(128) uint8_t smem[];
     constexpr int BQ = RG * 16;
     const int NC = DK / 8;                    // 16-byte chunks of a row
@@ -77,6 +79,8 @@ attention_latent_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
     const int pairs = min(BQ, len * H - pair0);
     const int tok0 = entry_start[e], pos0 = entry_pos0[e];
     const int pos_last = pos0 + (pair0 + pairs - 1) / H;
+    // the first key any query of the tile sees
+    const int key_first = window > 0 ? max(0, pos0 + pair0 / H - window + 1) : 0;
     const int* bt = block_table + (size_t)e * max_blocks;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, threads = blockDim.x;
     const int g = lane >> 2, t4 = lane & 3;
@@ -97,7 +101,7 @@ attention_latent_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
         if (tid < BKV) {
             const int key = kb + tid;
             int page = -1;
-            if (key <= pos_last) {
+            if (key <= pos_last && key >= key_first) {
                 const int blk = key / P;
                 page = blk < max_blocks ? bt[blk] : -1;
                 if (page < 0 || page >= n_pages) {
@@ -118,16 +122,19 @@ attention_latent_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
         }
     };
     // this split's share of the key tiles
-    const int all_tiles = pos_last / BKV + 1;
-    const int per_split = (all_tiles + n_splits - 1) / n_splits;
-    const int tile_lo = blockIdx.y * per_split, tile_hi = min(all_tiles, tile_lo + per_split);
+    const int tile_0 = key_first / BKV, all_tiles = pos_last / BKV + 1;
+    const int per_split = (all_tiles - tile_0 + n_splits - 1) / n_splits;
+    const int tile_lo = tile_0 + blockIdx.y * per_split, tile_hi = min(all_tiles, tile_lo + per_split);
 
     float o[2 * VT][4], m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
 #pragma unroll
     for (int i = 0; i < 2 * VT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-    int qpos[2];
+    int qpos[2], qlow[2];                    // a row's position, and the last key its window no longer covers
 #pragma unroll
-    for (int i = 0; i < 2; ++i) qpos[i] = pos0 + (pair0 + rg * 16 + g + 8 * i) / H;
+    for (int i = 0; i < 2; ++i) {
+        qpos[i] = pos0 + (pair0 + rg * 16 + g + 8 * i) / H;
+        qlow[i] = window > 0 ? qpos[i] - window : -1;
+    }
     const int mi = lane >> 3;
     const uint32_t q_frag = smem_addr(sQ + (rg * 16 + (mi & 1) * 8 + (lane & 7)) * RB + (mi >> 1) * 16);
     const uint32_t k_frag = (uint32_t)(((mi >> 1) * 8 + (lane & 7)) * RB + (mi & 1) * 16);
@@ -171,7 +178,7 @@ attention_latent_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
             for (int i = 0; i < 4; ++i) {
                 const int key = kb + nt * 8 + 2 * t4 + (i & 1);
                 float v = s[nt][i] * scale_log2e;
-                if (key > qpos[i >> 1]) v = -CUDART_INF_F;
+                if (key > qpos[i >> 1] || key <= qlow[i >> 1]) v = -CUDART_INF_F;
                 s[nt][i] = v;
                 mx[i >> 1] = fmaxf(mx[i >> 1], v);
             }
@@ -269,6 +276,7 @@ attention_latent_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
             const float keep = m[r] == -CUDART_INF_F ? 0.f : exp2f(m[r] - m2);
             inv = keep / (l[r] * keep + exp2f(s2 - m2));
         }
+        if (gate) inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)tok * gate_stride + h])));
         __nv_bfloat16* dst = out + (size_t)tok * out_stride + (size_t)h * DV + 2 * t4;
 #pragma unroll
         for (int i = 0; i < 2 * VT; ++i) {
@@ -283,7 +291,7 @@ attention_latent_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
 __global__ void __launch_bounds__(128)
 attention_latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                               __nv_bfloat16* __restrict__ out, int out_stride, int n_tokens, int H, int DV, int n_splits,
-                              const float* __restrict__ sink) {
+                              const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int gate_stride) {
     dd_launch_dependents();
     dd_grid_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -303,6 +311,7 @@ attention_latent_merge_kernel(const float* __restrict__ part_o, const float* __r
     for (int d = 16; d > 0; d >>= 1) total += __shfl_xor_sync(0xffffffffu, total, d);
     if (sink) total += exp2f(s2 - mx);
     w *= total > 0.f ? 1.f / total : 0.f;
+    if (gate) w *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)t * gate_stride + h])));
     const float* po = part_o + (size_t)row * n_splits * DV;
     __nv_bfloat16* dst = out + (size_t)t * out_stride + (size_t)h * DV;
     for (int c0 = 0; c0 < DV; c0 += 128) {   // (every lane walks the loop: the weights travel by shuffles)
@@ -328,7 +337,7 @@ attention_latent_merge_kernel(const float* __restrict__ part_o, const float* __r
 constexpr int PM = 64, PN = 128, PK = 32, PRB = PK * 2 + 16;
 __global__ void __launch_bounds__(128)
 per_head_mma_kernel(const __nv_bfloat16* __restrict__ in, int in_stride, int in_head, const __nv_bfloat16* __restrict__ w,
-                    __nv_bfloat16* __restrict__ out, int out_stride, int out_head, int n, int I, int J, int tail) {
+                    __nv_bfloat16* __restrict__ out, int out_stride, int out_head, int n, int I, int J, int tail, DdTailTurn turn) {
     __shared__ __align__(128) uint8_t sA[2][PM * PRB];
     __shared__ __align__(128) uint8_t sB[2][PN * PRB];
     dd_launch_dependents();
@@ -393,17 +402,15 @@ per_head_mma_kernel(const __nv_bfloat16* __restrict__ in, int in_stride, int in_
         }
     }
     if (tail > 0 && blockIdx.z == 0)
-        for (int idx = tid; idx < PM * tail; idx += 128) {
-            const int t = t0 + idx / tail, c = idx % tail;
-            if (t < n) out[(size_t)t * out_stride + (size_t)h * out_head + J + c] = in[(size_t)t * in_stride + (size_t)h * in_head + I + c];
-        }
+        dd_copy_tail<__nv_bfloat16>(in + (size_t)t0 * in_stride + (size_t)h * in_head + I, in_stride,
+                                    out + (size_t)t0 * out_stride + (size_t)h * out_head + J, out_stride, min(PM, n - t0), tail, t0, turn, 128);
 }
 
 template <int VT, int RG>
 int launch_latent(const void* q, int q_stride, const void* cache, const int* entry_start, const int* entry_pos0, int n_entries,
                   int n_tokens, const int* block_table, int max_blocks, void* out, int out_stride, float* part_o,
                   float* part_ml, int H, int DK, int DV, int P, int n_pages, float scale, int n_splits, int* error_flag,
-                  const float* sink, cudaStream_t s) {
+                  const float* sink, int window, const void* gate, int gate_stride, cudaStream_t s) {
     constexpr int BQ = RG * 16;
     // two key buffers, unless only one lets two blocks share an SM: with a warp a scheduler the tensor pipe idles most
     // of the time (measured: 17% active), and a second block fills more of it than a block's own prefetch
@@ -421,7 +428,8 @@ int launch_latent(const void* q, int q_stride, const void* cache, const int* ent
     dim3 grid(dd_ceil_div((long long)n_tokens * H, BQ) + n_entries, n_splits);
     dd_launch(attention_latent_kernel<VT, RG>, grid, dim3(32 * RG * slices), (size_t)smem, s, (const __nv_bfloat16*)q, q_stride,
               (const __nv_bfloat16*)cache, entry_start, entry_pos0, n_entries, block_table, max_blocks, (__nv_bfloat16*)out,
-              out_stride, part_o, part_ml, H, DK, DV, P, n_pages, scale * 1.4426950408889634f, n_splits, error_flag, sink, n_bufs);
+              out_stride, part_o, part_ml, H, DK, DV, P, n_pages, scale * 1.4426950408889634f, n_splits, error_flag, sink, n_bufs,
+              window, (const __nv_bfloat16*)gate, gate_stride);
     return dd_check_launch("dd_attention_latent");
 }
 }  // namespace
@@ -437,12 +445,16 @@ DD_API int dd_attention_latent_tile(int n_tokens, int n_entries, int H) { return
 
 // q: [N, q_stride] rows of H * DK; cache: [n_pages, P * DK]; entries are runs of consecutive tokens of one request
 // (entry_start [E+1], entry_pos0 [E], block_table row e). out: [N, out_stride] rows of H * DV. part_o
-// [N * H * n_splits * DV] and part_ml [N * H * n_splits * 2] only with n_splits > 1. Error bit 2: a key without a page.
+// [N * H * n_splits * DV] and part_ml [N * H * n_splits * 2] only with n_splits > 1. window > 0: a token sees itself and the
+// window - 1 keys before it. gate: [N, gate_stride] bfloat16 rows with one element per head, or null: a head's result is
+// multiplied by its logistic function. Error bit 2: a key without a page.
 DD_API int dd_attention_latent(const void* q, int q_stride, const void* cache, const int* entry_start, const int* entry_pos0,
                                int n_entries, int n_tokens, const int* block_table, int max_blocks, void* out, int out_stride,
                                float* part_o, float* part_ml, int H, int DK, int DV, int P, int n_pages, float scale,
-                               int n_splits, int* error_flag, const float* sink, void* stream) {
+                               int n_splits, int* error_flag, const float* sink, void* stream, int window, const void* gate,
+                               int gate_stride) {
     if (n_tokens <= 0 || n_entries <= 0) return 0;
+    if (window < 0) return dd_fail("dd_attention_latent: window %d must not be negative", window);
     if (!dd_attention_latent_supported(DK, DV, DD_BF16))
         return dd_fail("dd_attention_latent: rows of %d with values of %d are not supported", DK, DV);
     if (q_stride % 8 || out_stride % 2 || ((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 3))
@@ -451,7 +463,7 @@ DD_API int dd_attention_latent(const void* q, int q_stride, const void* cache, c
     cudaStream_t s = (cudaStream_t)stream;
     int rc;
 #define DD_LATENT(VT, RG) launch_latent<VT, RG>(q, q_stride, cache, entry_start, entry_pos0, n_entries, n_tokens, block_table, max_blocks, \
-                                        out, out_stride, part_o, part_ml, H, DK, DV, P, n_pages, scale, n_splits, error_flag, sink, s)
+                                        out, out_stride, part_o, part_ml, H, DK, DV, P, n_pages, scale, n_splits, error_flag, sink, window, gate, gate_stride, s)
     if (dd_attention_latent_tile(n_tokens, n_entries, H) == 32) {
         // single tokens: more warps with fewer value columns each (both slices of a row compute its scores)
         if (DV <= 64) rc = DD_LATENT(4, 2);
@@ -462,7 +474,7 @@ DD_API int dd_attention_latent(const void* q, int q_stride, const void* cache, c
 #undef DD_LATENT
     if (rc || n_splits == 1) return rc;
     dd_launch(attention_latent_merge_kernel, dim3(dd_ceil_div((long long)n_tokens * H, 4)), dim3(128), 0, s, (const float*)part_o,
-              (const float*)part_ml, (__nv_bfloat16*)out, out_stride, n_tokens, H, DV, n_splits, sink);
+              (const float*)part_ml, (__nv_bfloat16*)out, out_stride, n_tokens, H, DV, n_splits, sink, (const __nv_bfloat16*)gate, gate_stride);
     return dd_check_launch("dd_attention_latent (merge)");
 }
 
@@ -471,13 +483,16 @@ DD_API int dd_per_head_mma_supported(int in_stride, int in_head, int out_stride,
 }
 
 DD_API int dd_per_head_mma(const void* in, int in_stride, int in_head, const void* w, void* out, int out_stride, int out_head,
-                           int n, int heads, int I, int J, int tail, void* stream) {
+                           int n, int heads, int I, int J, int tail, void* stream, const float* freqs, int n_pairs, int interleaved,
+                           const int* positions) {
     if (n <= 0 || heads <= 0) return 0;
+    if (n_pairs < 0 || 2 * n_pairs > tail || (n_pairs > 0 && (!freqs || !positions))) return dd_fail("dd_per_head_mma: %d pairs do not fit a tail of %d", n_pairs, tail);
+    const DdTailTurn turn = {freqs, positions, n_pairs, interleaved};
     if (J <= 0 || tail < 0 || heads > 65535 || !dd_per_head_mma_supported(in_stride, in_head, out_stride, out_head, I, DD_BF16))
         return dd_fail("dd_per_head_mma: sizes are not supported");
     if (((uintptr_t)in & 15) || ((uintptr_t)w & 15) || ((uintptr_t)out & 3)) return dd_fail("dd_per_head_mma: rows must be 16-byte aligned");
     dd_launch(per_head_mma_kernel, dim3(dd_ceil_div(n, PM), heads, dd_ceil_div(J, PN)), dim3(128), 0, (cudaStream_t)stream,
               (const __nv_bfloat16*)in, in_stride, in_head, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_stride, out_head,
-              n, I, J, tail);
+              n, I, J, tail, turn);
     return dd_check_launch("dd_per_head_mma");
 }

@@ -9,7 +9,7 @@
 #define DD_API extern "C" __attribute__((visibility("default")))
 
 enum DdDtype { DD_F32 = 0, DD_BF16 = 1 };
-enum DdAct { DD_ACT_NONE = 0, DD_ACT_GELU_NEW = 1, DD_ACT_GELU_ERF = 2, DD_ACT_RELU2 = 3 };
+enum DdAct { DD_ACT_NONE = 0, DD_ACT_GELU_NEW = 1, DD_ACT_GELU_ERF = 2, DD_ACT_RELU2 = 3, DD_ACT_TANH = 4 };
 
 // Records a message for dd_last_error() and returns a non-zero code.
 int dd_fail(const char* fmt, ...);
@@ -38,7 +38,7 @@ __device__ __forceinline__ float dd_warp_max(float v) {
 }
 
 // gelu_new(u) = 0.5 u (1 + tanh(sqrt(2/pi) (u + 0.044715 u^3))); gelu(u) = 0.5 u (1 + erf(u / sqrt 2));
-// relu2(u) = max(u, 0)^2.
+// relu2(u) = max(u, 0)^2; tanh.
 __device__ __forceinline__ float dd_activation(float u, int act) {
     if (act == DD_ACT_GELU_NEW) {
         const float c = 0.7978845608028654f;
@@ -46,6 +46,7 @@ __device__ __forceinline__ float dd_activation(float u, int act) {
     }
     if (act == DD_ACT_GELU_ERF) return 0.5f * u * (1.0f + erff(u * 0.7071067811865476f));
     if (act == DD_ACT_RELU2) { const float r = fmaxf(u, 0.f); return r * r; }
+    if (act == DD_ACT_TANH) return tanhf(u);
     return u;
 }
 
@@ -60,6 +61,34 @@ __device__ __forceinline__ float dd_gated_value(float gate, float up, int form, 
     const float g = fminf(gate, limit);
     const float u = fminf(fmaxf(up, -limit), limit);
     return g * (1.0f / (1.0f + (FAST ? __expf(-alpha * g) : expf(-alpha * g)))) * (u + 1.0f);
+}
+
+// A rotation that `tail` elements undergo while they are copied: n_pairs pairs (neighbours, or one of each half of the first
+// 2 * n_pairs elements) turned by positions[token] * freqs[pair], float32 inside; n_pairs = 0: a plain copy.
+struct DdTailTurn {
+    const float* freqs;
+    const int* positions;
+    int n_pairs, interleaved;
+};
+// Copies the tails of `n` consecutive rows (the first is token t0) by a block's threads.
+template <typename T>
+__device__ __forceinline__ void dd_copy_tail(const T* in, int in_stride, T* out, int out_stride, int n, int tail, int t0,
+                                             const DdTailTurn& turn, int threads) {
+    if (turn.n_pairs > 0)
+        for (int i = threadIdx.x; i < n * turn.n_pairs; i += threads) {
+            const int tt = i / turn.n_pairs, p = i % turn.n_pairs;
+            const int c = turn.interleaved ? 2 * p : p, to = turn.interleaved ? 1 : turn.n_pairs;
+            float sn, cs;
+            sincosf((float)turn.positions[t0 + tt] * turn.freqs[p], &sn, &cs);
+            const float a = dd_to_f32(in[(size_t)tt * in_stride + c]), b = dd_to_f32(in[(size_t)tt * in_stride + c + to]);
+            out[(size_t)tt * out_stride + c] = dd_from_f32<T>(a * cs - b * sn);
+            out[(size_t)tt * out_stride + c + to] = dd_from_f32<T>(b * cs + a * sn);
+        }
+    const int rest = tail - 2 * turn.n_pairs;
+    for (int i = threadIdx.x; i < n * rest; i += threads) {
+        const int tt = i / rest, c = 2 * turn.n_pairs + i % rest;
+        out[(size_t)tt * out_stride + c] = in[(size_t)tt * in_stride + c];
+    }
 }
 
 static inline int dd_ceil_div(long long a, long long b) { return (int)((a + b - 1) / b); }

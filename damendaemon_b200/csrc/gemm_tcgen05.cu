@@ -134,6 +134,7 @@ __device__ __forceinline__ void store16(const GemmParams& p, int m_first, int n,
             } else v = dd_activation(v, DD_ACT_GELU_NEW);
         } else if (ACT == DD_ACT_GELU_ERF) v = dd_activation(v, DD_ACT_GELU_ERF);
         else if (ACT == DD_ACT_RELU2) v = dd_activation(v, DD_ACT_RELU2);
+        else if (ACT == DD_ACT_TANH) v = dd_activation(v, DD_ACT_TANH);
         if (RESIDUAL) v += r[j];
         if (BF16_OUT) reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)(m_first + j) * p.ldo + n] = __float2bfloat16_rn(v);
         else reinterpret_cast<float*>(p.out)[(size_t)(m_first + j) * p.ldo + n] = v;
@@ -164,6 +165,7 @@ __device__ __forceinline__ void store_out16(const GemmParams& p, int m_first, in
     if (p.act == DD_ACT_NONE) store16_o<DD_ACT_NONE>(p, m_first, n, acc, b, r);
     else if (p.act == DD_ACT_GELU_NEW) store16_o<DD_ACT_GELU_NEW>(p, m_first, n, acc, b, r);
     else if (p.act == DD_ACT_RELU2) store16_o<DD_ACT_RELU2>(p, m_first, n, acc, b, r);
+    else if (p.act == DD_ACT_TANH) store16_o<DD_ACT_TANH>(p, m_first, n, acc, b, r);
     else store16_o<DD_ACT_GELU_ERF>(p, m_first, n, acc, b, r);
 }
 
@@ -226,6 +228,7 @@ __device__ __forceinline__ void store_row16(const GemmParams& p, int m, int n_fi
             } else u = dd_activation(u, DD_ACT_GELU_NEW);
         } else if (ACT == DD_ACT_GELU_ERF) u = dd_activation(u, DD_ACT_GELU_ERF);
         else if (ACT == DD_ACT_RELU2) u = dd_activation(u, DD_ACT_RELU2);
+        else if (ACT == DD_ACT_TANH) u = dd_activation(u, DD_ACT_TANH);
         if (RESIDUAL) u += r[j];
         v[j] = u;
     }
@@ -278,6 +281,7 @@ __device__ __forceinline__ void store_out_row16(const GemmParams& p, int m, int 
     if (p.act == DD_ACT_NONE) store_row16_o<DD_ACT_NONE>(p, m, n_first, acc, r, v);
     else if (p.act == DD_ACT_GELU_NEW) store_row16_o<DD_ACT_GELU_NEW>(p, m, n_first, acc, r, v);
     else if (p.act == DD_ACT_RELU2) store_row16_o<DD_ACT_RELU2>(p, m, n_first, acc, r, v);
+    else if (p.act == DD_ACT_TANH) store_row16_o<DD_ACT_TANH>(p, m, n_first, acc, r, v);
     else store_row16_o<DD_ACT_GELU_ERF>(p, m, n_first, acc, r, v);
 }
 

@@ -4,17 +4,20 @@
 // which every expert's rows start on a multiple of the product's row tile, so that a tile of rows meets one
 // expert's matrices only (tile_group[tile] = that expert, or -1 for a tile no pair fell into):
 //
-//   dd_route_by_table   token ids + table [vocab, K] -> pair_row [N*K] (the row of pair (t, k)), row_token [rows]
+//   dd_route_by_table   token ids + table [vocab, K] -> pair_row [N*K] (the row of pair (t, k); -2 for an
+//                       identity expert, whose output is the token's own input row: experts n_experts .. n_experts +
+//                       n_identity - 1 of the table; they have no rows), row_token [rows]
 //                       (the token of a row, -1 for a row of padding), tile_group [rows / tile]
 //   dd_gather_rows      x [N, width] -> sorted rows (a row of padding is zeroed)
 //                       (ids null: token t reads row t of the table, which then holds the step's own choices)
 //   dd_route_by_score   normed rows [N, width] and the router's matrix -> float32 logits, then the K experts of every token
-//                       by score within the worthiest groups, their weights, and the gate of a shared unit
+//                       by score (sigmoid, or softmax over all; a correction per expert may move the choice) within the
+//                       worthiest groups, their weights (as scored, or divided by their sum), and the gate of a shared unit
 //   dd_gated_unit       rows of [gate | up] halves -> y = f(gate, up) in float32 (dd_gated_value in common.cuh: the
 //                       clamped form g * sigmoid(alpha g) * (u + 1), silu(gate) * up, or tanh-gelu(gate) * up),
 //                       optionally times a number per row
 //   dd_combine_rows     stream[t] += sum over k of weight (* pair_weight[t*K + k]) * y[pair_row[t*K + k]], k ascending,
-//                       in float32
+//                       in float32; own[t] in place of a row of y where pair_row is -2
 //
 // The order of an expert's rows among themselves depends on the order in which threads arrive; no value depends
 // on it, since every row is computed by itself and the sum over a token's experts runs in the order of its choices.
@@ -26,7 +29,7 @@ constexpr int ROUTE_THREADS = 1024;
 __global__ void __launch_bounds__(ROUTE_THREADS)
 route_by_table_kernel(const int* __restrict__ ids, const int* __restrict__ table, int n_tokens, int vocab, int top,
                       int n_experts, int tile, int n_rows, int* __restrict__ pair_row, int* __restrict__ row_token,
-                      int* __restrict__ tile_group, int* __restrict__ error_flag) {
+                      int* __restrict__ tile_group, int* __restrict__ error_flag, int n_identity) {
     extern __shared__ int shared[];              // [E] counts, then cursors; [E + 1] first rows
     int* count = shared;
     int* first = shared + n_experts;
@@ -50,7 +53,7 @@ route_by_table_kernel(const int* __restrict__ ids, const int* __restrict__ table
         for (int u = 0; u < 4; ++u) {
             const int pair = base + u * ROUTE_THREADS;
             e[u] = (id[u] >= 0 && id[u] < vocab) ? table[(size_t)id[u] * top + pair % top] : -1;
-            if (e[u] >= n_experts) e[u] = -1;
+            if (e[u] < 0 || e[u] >= n_experts) e[u] = (e[u] >= n_experts && e[u] < n_experts + n_identity) ? -2 : -1;
         }
     };
     for (int base = threadIdx.x; base < n_pairs; base += 4 * ROUTE_THREADS) {
@@ -59,8 +62,8 @@ route_by_table_kernel(const int* __restrict__ ids, const int* __restrict__ table
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
             if (base + u * ROUTE_THREADS >= n_pairs) break;
-            if (e[u] < 0) atomicOr(error_flag, 1);
-            else atomicAdd(&count[e[u]], 1);
+            if (e[u] == -1) atomicOr(error_flag, 1);
+            else if (e[u] >= 0) atomicAdd(&count[e[u]], 1);
         }
     }
     __syncthreads();
@@ -84,7 +87,7 @@ route_by_table_kernel(const int* __restrict__ ids, const int* __restrict__ table
             const int pair = base + u * ROUTE_THREADS;
             if (pair >= n_pairs) break;
             if (e[u] < 0) {
-                pair_row[pair] = -1;
+                pair_row[pair] = e[u];           // -2: the token's own row
                 continue;
             }
             const int row = first[e[u]] + atomicAdd(&count[e[u]], 1);
@@ -127,15 +130,17 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 route_by_score_kernel(const T* __restrict__ y, int ldy, const T* __restrict__ router, int ldr, int width, int n_tokens,
                       int n_experts, int top, int groups, int keep, float weight_scale, int gate_row,
-                      int* __restrict__ chosen, float* __restrict__ pair_weight, float* __restrict__ shared_scale) {
-    extern __shared__ float route_smem[];        // [E] scores, [groups] worths, [4][rows] the warps' sums
+                      int* __restrict__ chosen, float* __restrict__ pair_weight, float* __restrict__ shared_scale,
+                      int softmax, const float* __restrict__ correction, int renormalize) {
+    extern __shared__ float route_smem[];        // [E] choice scores, [E] scores, [groups] worths, [4][rows] the warps' sums
     dd_launch_dependents();
     dd_grid_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
     const int n_rows = n_experts + (gate_row >= 0 ? 1 : 0);          // the shared unit's gate vector is one more row
-    float* score = route_smem;
-    float* worth = score + n_experts;
+    float* score = route_smem;                   // what the choice looks at
+    float* value = score + n_experts;            // what a chosen expert weighs
+    float* worth = value + n_experts;
     float* part = worth + groups;
     const T* x = y + (size_t)t * ldy;
     constexpr int V = RoutePiece<T>::N, ROWS = 17;       // sixteen experts and a shared unit's gate in one pass
@@ -174,18 +179,38 @@ route_by_score_kernel(const T* __restrict__ y, int ldy, const T* __restrict__ ro
     __syncthreads();
     for (int e = threadIdx.x; e < n_rows; e += 128) {
         const float z = ((part[e] + part[n_rows + e]) + part[2 * n_rows + e]) + part[3 * n_rows + e];
+        if (e < n_experts && softmax) {
+            value[e] = z;                        // the logits; the first warp turns them into scores
+            continue;
+        }
         const float s = 1.0f / (1.0f + expf(-z));
-        if (e < n_experts) score[e] = s;
-        else if (shared_scale) shared_scale[t] = s;
+        if (e < n_experts) {
+            value[e] = s;
+            score[e] = correction ? s + correction[e] : s;
+        } else if (shared_scale) shared_scale[t] = s;
     }
     if (threadIdx.x == 0 && shared_scale && gate_row < 0) shared_scale[t] = 1.0f;
     __syncthreads();
     if (warp) return;
     __syncwarp();
+    constexpr float NONE = -3.0e38f;             // below every score: struck out
+    if (softmax) {
+        float top_z = NONE, total = 0.f;
+        for (int e = lane; e < n_experts; e += 32) top_z = fmaxf(top_z, value[e]);
+        top_z = dd_warp_max(top_z);
+        for (int e = lane; e < n_experts; e += 32) total += expf(value[e] - top_z);
+        total = dd_warp_sum(total);
+        for (int e = lane; e < n_experts; e += 32) {
+            const float s = expf(value[e] - top_z) / total;
+            value[e] = s;
+            score[e] = correction ? s + correction[e] : s;
+        }
+        __syncwarp();
+    }
     const int per = n_experts / groups;
     if (groups > 1) {
         for (int g = lane; g < groups; g += 32) {
-            float best = -1.f, second = -1.f;            // scores lie in [0, 1]
+            float best = NONE, second = NONE;
             for (int i = 0; i < per; ++i) {
                 const float s = score[g * per + i];
                 if (s > best) { second = best; best = s; }
@@ -195,25 +220,27 @@ route_by_score_kernel(const T* __restrict__ y, int ldy, const T* __restrict__ ro
         }
         __syncwarp();
         // keep the worthiest runs: the others' scores are struck out
+        // (a kept run's worth becomes infinite and is passed over from then on)
         for (int round = 0; round < keep; ++round) {
-            float best = -1.f;
+            float best = -INFINITY;
             int at = 0x7fffffff;
             for (int g = lane; g < groups; g += 32)
-                if (worth[g] > best) { best = worth[g]; at = g; }
+                if (worth[g] > best && worth[g] < INFINITY) { best = worth[g]; at = g; }
             for (int o = 16; o > 0; o >>= 1) {
                 const float ob = __shfl_xor_sync(0xffffffffu, best, o);
                 const int oa = __shfl_xor_sync(0xffffffffu, at, o);
                 if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
             }
-            if (lane == 0 && at < groups) worth[at] = -2.f;     // marked as kept
+            if (lane == 0 && at < groups) worth[at] = INFINITY;     // marked as kept
             __syncwarp();
         }
         for (int e = lane; e < n_experts; e += 32)
-            if (worth[e / per] != -2.f) score[e] = -1.f;
+            if (worth[e / per] != INFINITY) score[e] = NONE;
         __syncwarp();
     }
+    float sum = 0.f;                             // of the chosen scores, in the order of the choice (lane 0)
     for (int k = 0; k < top; ++k) {
-        float best = -1.f;
+        float best = NONE;
         int at = 0x7fffffff;
         for (int e = lane; e < n_experts; e += 32)
             if (score[e] > best) { best = score[e]; at = e; }
@@ -224,11 +251,15 @@ route_by_score_kernel(const T* __restrict__ y, int ldy, const T* __restrict__ ro
         }
         if (lane == 0) {
             chosen[(size_t)t * top + k] = at < n_experts ? at : -1;
-            pair_weight[(size_t)t * top + k] = at < n_experts ? best * weight_scale : 0.f;
-            if (at < n_experts) score[at] = -1.f;
+            const float s = at < n_experts ? value[at] : 0.f;
+            pair_weight[(size_t)t * top + k] = s * weight_scale;
+            sum += s;
+            if (at < n_experts) score[at] = NONE;
         }
         __syncwarp();
     }
+    if (renormalize && lane == 0)
+        for (int k = 0; k < top; ++k) pair_weight[(size_t)t * top + k] /= sum + 1e-20f;
 }
 
 template <typename T>
@@ -282,9 +313,10 @@ gated_unit_kernel(const T* __restrict__ gate_up, int stride, T* __restrict__ out
     }
 }
 
+template <typename T>
 __global__ void __launch_bounds__(128)
 combine_rows_kernel(const float* __restrict__ y, const int* __restrict__ pair_row, float* __restrict__ stream, int width,
-                    int top, float weight, const float* __restrict__ pair_weight) {
+                    int top, float weight, const float* __restrict__ pair_weight, const T* __restrict__ own) {
     dd_launch_dependents();
     dd_grid_wait();
     const int t = blockIdx.x;
@@ -308,6 +340,11 @@ combine_rows_kernel(const float* __restrict__ y, const int* __restrict__ pair_ro
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
             v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (row[u] == -2 && own) {           // the token's own row
+                const T* src = own + (size_t)t * width + c;
+                v[u].x = dd_to_f32(src[0]);
+                if (wide) { v[u].y = dd_to_f32(src[1]); v[u].z = dd_to_f32(src[2]); v[u].w = dd_to_f32(src[3]); }
+            }
             if (row[u] < 0) continue;
             const float* src = y + (size_t)row[u] * width + c;
             if (wide) v[u] = *reinterpret_cast<const float4*>(src);
@@ -333,7 +370,8 @@ combine_rows_kernel(const float* __restrict__ y, const int* __restrict__ pair_ro
 // n_rows: rows of the sorted buffer, a multiple of tile and at least n_tokens * top + min(n_experts, n_tokens * top)
 // * (tile - 1): every expert that has a pair may waste all but one row of its last tile. A token id or a table entry out of range sets error bit 1 and leaves its pair out.
 DD_API int dd_route_by_table(const int* ids, const int* table, int n_tokens, int vocab, int top, int n_experts, int tile,
-                             int n_rows, int* pair_row, int* row_token, int* tile_group, int* error_flag, void* stream) {
+                             int n_rows, int* pair_row, int* row_token, int* tile_group, int* error_flag, void* stream,
+                             int n_identity) {
     if (n_tokens <= 0) return 0;
     const long long n_pairs = (long long)n_tokens * top;
     if (top <= 0 || n_experts <= 0 || tile <= 0 || n_rows % tile ||
@@ -342,7 +380,7 @@ DD_API int dd_route_by_table(const int* ids, const int* table, int n_tokens, int
                        n_tokens, top, n_experts);
     if (n_experts > 8192) return dd_fail("dd_route_by_table: %d experts are more than a block counts", n_experts);
     dd_launch(route_by_table_kernel, dim3(1), dim3(ROUTE_THREADS), (size_t)(2 * n_experts + 1) * sizeof(int), (cudaStream_t)stream,
-              ids, table, n_tokens, vocab, top, n_experts, tile, n_rows, pair_row, row_token, tile_group, error_flag);
+              ids, table, n_tokens, vocab, top, n_experts, tile, n_rows, pair_row, row_token, tile_group, error_flag, n_identity);
     return dd_check_launch("dd_route_by_table");
 }
 
@@ -352,24 +390,28 @@ DD_API int dd_route_by_table(const int* ids, const int* table, int n_tokens, int
 // `keep` worthiest runs stay eligible; the `top` largest eligible scores win. chosen: int32 [n_tokens, top] by falling
 // score (-1 where fewer were eligible), pair_weight: float32 [n_tokens, top] = score * weight_scale. shared_scale (or
 // null): float32 [n_tokens] = sigmoid(y . router row gate_row), 1 with gate_row < 0 (gate_row is n_experts or negative).
+// softmax: scores are the softmax of the n_experts logits instead. correction (float32 [n_experts] or null) is added to the
+// scores for the choice only. renormalize: the chosen weights are divided by (the sum of the chosen scores + 1e-20).
 DD_API int dd_route_by_score(const void* y, int ldy, const void* router, int ldr, int width, int n_tokens, int n_experts,
                              int top, int groups, int keep, float weight_scale, int gate_row, int* chosen,
-                             float* pair_weight, float* shared_scale, int dtype, void* stream) {
+                             float* pair_weight, float* shared_scale, int dtype, void* stream, int softmax,
+                             const float* correction, int renormalize) {
     if (n_tokens <= 0) return 0;
     if (n_experts <= 0 || top <= 0 || top > n_experts || groups <= 0 || n_experts % groups || keep <= 0 || keep > groups ||
         (gate_row >= 0 && gate_row != n_experts) || width <= 0)
         return dd_fail("dd_route_by_score: %d of %d experts in %d groups of which %d stay, gate row %d", top, n_experts, groups, keep, gate_row);
-    const size_t smem = (size_t)(n_experts + groups + 4 * (n_experts + 1)) * sizeof(float);
+    const size_t smem = (size_t)(2 * n_experts + groups + 4 * (n_experts + 1)) * sizeof(float);
     if (smem > 48 * 1024) return dd_fail("dd_route_by_score: %d experts are more than a block's shared memory holds", n_experts);
     cudaStream_t s = (cudaStream_t)stream;
     const dim3 grid(n_tokens);
     if (dtype == DD_F32)
         dd_launch(route_by_score_kernel<float>, grid, dim3(128), smem, s, (const float*)y, ldy, (const float*)router, ldr, width,
-                  n_tokens, n_experts, top, groups, keep, weight_scale, gate_row, chosen, pair_weight, shared_scale);
+                  n_tokens, n_experts, top, groups, keep, weight_scale, gate_row, chosen, pair_weight, shared_scale, softmax,
+                  correction, renormalize);
     else if (dtype == DD_BF16)
         dd_launch(route_by_score_kernel<__nv_bfloat16>, grid, dim3(128), smem, s, (const __nv_bfloat16*)y, ldy,
                   (const __nv_bfloat16*)router, ldr, width, n_tokens, n_experts, top, groups, keep, weight_scale, gate_row, chosen,
-                  pair_weight, shared_scale);
+                  pair_weight, shared_scale, softmax, correction, renormalize);
     else
         return dd_fail("dd_route_by_score: unknown dtype %d", dtype);
     return dd_check_launch("dd_route_by_score");
@@ -410,10 +452,16 @@ DD_API int dd_gated_unit(const void* gate_up, int stride, void* out, int out_str
 }
 
 DD_API int dd_combine_rows(const float* y, const int* pair_row, float* stream_rows, int n_tokens, int width, int top,
-                           float weight, void* stream, const float* pair_weight) {
+                           float weight, void* stream, const float* pair_weight, const void* own, int own_dtype) {
     if (n_tokens <= 0) return 0;
+    if (own && own_dtype != DD_F32 && own_dtype != DD_BF16) return dd_fail("dd_combine_rows: unknown dtype %d", own_dtype);
     const bool wide = width % 4 == 0 && !(((uintptr_t)y | (uintptr_t)stream_rows) & 15);
-    dd_launch(combine_rows_kernel, dim3(n_tokens, dd_ceil_div(width, wide ? 512 : 128)), dim3(128), 0, (cudaStream_t)stream, y, pair_row,
-              stream_rows, width, top, weight, pair_weight);
+    const dim3 grid(n_tokens, dd_ceil_div(width, wide ? 512 : 128));
+    if (own && own_dtype == DD_F32)
+        dd_launch(combine_rows_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, y, pair_row, stream_rows, width, top, weight,
+                  pair_weight, (const float*)own);
+    else
+        dd_launch(combine_rows_kernel<__nv_bfloat16>, grid, dim3(128), 0, (cudaStream_t)stream, y, pair_row, stream_rows, width, top,
+                  weight, pair_weight, (const __nv_bfloat16*)own);
     return dd_check_launch("dd_combine_rows");
 }

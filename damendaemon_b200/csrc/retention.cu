@@ -34,8 +34,8 @@
 // tokens' read-outs side by side (a token's state update depends on the token before, its read-out's sum on nothing
 // that follows).
 //
-// dd_retention_finish then divides every head's o by its root mean square (eps inside the root, no weight), multiplies
-// by silu(gate) and rounds to the storage type: the operand of the output projection.
+// dd_retention_finish then divides every head's o by its root mean square (eps inside the root; optionally a weight per
+// element), multiplies by silu(gate) and rounds to the storage type: the operand of the output projection.
 #include "common.cuh"
 
 namespace {
@@ -297,7 +297,7 @@ retention_prepare_kernel(const T* __restrict__ q, const T* __restrict__ k, const
 template <typename T, int PER>
 __global__ void __launch_bounds__(128)
 retention_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_stride, T* __restrict__ out,
-                        int out_stride, int n_tokens, int heads, int dv, float eps) {
+                        int out_stride, int n_tokens, int heads, int dv, float eps, const float* __restrict__ weight) {
     dd_launch_dependents();
     dd_grid_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -321,7 +321,7 @@ retention_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate,
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
         const int c = lane + 32 * i;
-        if (c < dv) dst[c] = dd_from_f32<T>(x[i] * r * (z[i] / (1.0f + expf(-z[i]))));
+        if (c < dv) dst[c] = dd_from_f32<T>(x[i] * r * (weight ? weight[h * dv + c] : 1.0f) * (z[i] / (1.0f + expf(-z[i]))));
     }
 }
 
@@ -412,15 +412,16 @@ DD_API int dd_retention(const void* q, const void* k, const void* v, int stride,
 }
 
 // o: float32 [tokens, heads * dv]; gate: rows of gate_stride elements with heads * dv values; out likewise (out_stride).
+// weight: float32 [heads * dv] that multiplies the normed read-out, or null.
 DD_API int dd_retention_finish(const float* o, const void* gate, int gate_stride, void* out, int out_stride, int n_tokens,
-                               int heads, int dv, float eps, int dtype, void* stream) {
+                               int heads, int dv, float eps, int dtype, void* stream, const float* weight) {
     if (n_tokens <= 0) return 0;
     if (dv <= 0 || dv > 1024) return dd_fail("dd_retention_finish: a value head of %d is not supported (at most 1024)", dv);
     cudaStream_t s = (cudaStream_t)stream;
     const int grid = dd_ceil_div((long long)n_tokens * heads, 4);
 #define DD_FINISH(T, PER)                                                                                                 \
     dd_launch(retention_finish_kernel<T, PER>, dim3(grid), dim3(128), 0, s, o, (const T*)gate, gate_stride, (T*)out, out_stride, \
-              n_tokens, heads, dv, eps)
+              n_tokens, heads, dv, eps, weight)
 #define DD_FINISH_SIZED(T)                                                     \
     do {                                                                       \
         if (dv <= 32) DD_FINISH(T, 1);                                         \

@@ -14,7 +14,7 @@ import torch
 from .csrc import build
 
 F32, BF16 = 0, 1
-ACTIVATIONS = {None: 0, "none": 0, "gelu_new": 1, "gelu": 2, "relu2": 3}
+ACTIVATIONS = {None: 0, "none": 0, "gelu_new": 1, "gelu": 2, "relu2": 3, "tanh": 4}
 GATED_FORMS = {"clamped_swish": 0, "silu": 1, "gelu_tanh": 2}     # the forms of a gated unit (csrc/common.cuh)
 
 _c_int, _c_float, _c_void = ctypes.c_int, ctypes.c_float, ctypes.c_void_p
@@ -41,20 +41,26 @@ _SIGNATURES = {
         "dd_delta_rule": [_c_void] * 7 + [_c_int, _c_void, _c_void] + [_c_int] * 4 + [_c_void],
         "dd_delta_finish": [_c_void] * 4 + [_c_int] * 4 + [_c_float, _c_int, _c_void],
         "dd_latent_prepare": [_c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_int, _c_void, _c_float, _c_void, _c_int,
-                              _c_void, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void],
-        "dd_per_head_linear": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int] + [_c_int] * 6 + [_c_void],
+                              _c_void, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void,
+                              _c_int, _c_void, _c_int, _c_int, _c_void, _c_void, _c_int],
+        "dd_per_head_linear": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int] + [_c_int] * 6 + [_c_void, _c_void, _c_int, _c_int, _c_void],
+        "dd_token_mix": [_c_void] * 4 + [_c_int] + [_c_void] * 7 + [ctypes.c_longlong, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void],
+        "dd_time_prepare": [_c_void, _c_void, _c_void, _c_int] + [_c_void] * 8 + [_c_int] * 5 + [_c_void],
+        "dd_time_scan": [_c_void] * 7 + [_c_int, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void],
+        "dd_time_step": [_c_void] * 4 + [_c_int] + [_c_void] * 4 + [_c_float, _c_void, _c_int, _c_void, _c_void] + [_c_int] * 5 + [_c_void],
         "dd_rotary": [_c_void, _c_void, _c_int, _c_void, _c_void, _c_float] + [_c_int] * 7 + [_c_void],
         "dd_gemm_simt_group_tile": [],
         "dd_gemm_simt_grouped": [_c_void, _c_int, _c_void, _c_int, ctypes.c_longlong, _c_void, _c_void, _c_int] + [_c_int] * 6 + [_c_void],
-        "dd_route_by_table": [_c_void, _c_void] + [_c_int] * 6 + [_c_void] * 5,
+        "dd_route_by_table": [_c_void, _c_void] + [_c_int] * 6 + [_c_void] * 5 + [_c_int],
         "dd_gather_rows": [_c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void],
         "dd_gated_unit": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void, _c_int, _c_void],
-        "dd_combine_rows": [_c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_float, _c_void, _c_void],
-        "dd_route_by_score": [_c_void, _c_int, _c_void, _c_int] + [_c_int] * 6 + [_c_float, _c_int, _c_void, _c_void, _c_void, _c_int, _c_void],
+        "dd_combine_rows": [_c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_float, _c_void, _c_void, _c_void, _c_int],
+        "dd_route_by_score": [_c_void, _c_int, _c_void, _c_int] + [_c_int] * 6 + [_c_float, _c_int, _c_void, _c_void, _c_void, _c_int, _c_void,
+                                                                                _c_int, _c_void, _c_int],
         "dd_head_norm_rotary": [_c_void, _c_void, _c_int, _c_void, _c_void, _c_void, _c_void, _c_float] + [_c_int] * 7 + [_c_void],
         "dd_retention": [_c_void, _c_void, _c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_void,
                          _c_float, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void],
-        "dd_retention_finish": [_c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void],
+        "dd_retention_finish": [_c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void, _c_void],
         "dd_gemm_simt": [_c_void, _c_int, _c_void, _c_int, _c_void, _c_void, _c_int, _c_void, _c_int] + [_c_int] * 6 + [_c_void],
         "dd_kv_store": [_c_void, _c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_void] + [_c_int] * 7 + [_c_void, _c_void],
         "dd_attention_rows": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_void, _c_int, _c_void, _c_int, _c_void, _c_void]
@@ -97,9 +103,9 @@ _SIGNATURES = {
         "dd_attention_latent_supported": [_c_int] * 3,
         "dd_attention_latent_tile": [_c_int] * 3,
         "dd_attention_latent": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int,
-                                _c_void, _c_void] + [_c_int] * 5 + [_c_float, _c_int, _c_void, _c_void, _c_void],
+                                _c_void, _c_void] + [_c_int] * 5 + [_c_float, _c_int, _c_void, _c_void, _c_void, _c_int, _c_void, _c_int],
         "dd_per_head_mma_supported": [_c_int] * 6,
-        "dd_per_head_mma": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int] + [_c_int] * 5 + [_c_void],
+        "dd_per_head_mma": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_int] + [_c_int] * 5 + [_c_void, _c_void, _c_int, _c_int, _c_void],
         "dd_attention_prefill_tcgen05_supported": [_c_int] * 5,
         "dd_attention_prefill_tcgen05": [_c_void, _c_int, _c_void, _c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int]
                                         + [_c_int] * 6 + [_c_float, _c_void, _c_void, _c_int, _c_void, _c_int],
@@ -657,34 +663,55 @@ def delta_finish(o, gate, weight, heads, eps, out_dtype, out=None):
     return out
 
 
-def latent_prepare(q, down, weight, eps, freqs, token_entry, positions, block_table, cache, heads, head_dim, rot_dim, rank):
+def latent_prepare(q, down, weight, eps, freqs, token_entry, positions, block_table, cache, heads, head_dim, rot_dim, rank,
+                   interleaved=True, second=None, second_weight=None):
     """A step's latent rows into the cache, and its queries rotated. down: [N, rank + rot_dim] row view; the cache row of a
     token becomes [rms(down[:rank]) * weight | down[rank:] rotated by its position] (cache [pages, page_size * (rank +
     rot_dim)]); the last rot_dim elements of every query head (q [N, heads * (head_dim + rot_dim)], a row view) are rotated
-    in place. Neighbouring dimensions pair; the first 2 * len(freqs) of the rot_dim turn. float32 inside."""
-    n = q.shape[0]
+    in place (q None: there are none yet). Neighbouring dimensions pair, or (interleaved False) the two halves; the first
+    2 * len(freqs) of the rot_dim turn. second: another row view [N, S] of down's type, divided by its root mean square
+    (the same eps) and multiplied by second_weight; returned as a tensor of its own (else None). float32 inside."""
+    n = down.shape[0]
     row = rank + rot_dim
-    if q.shape[1] != heads * (head_dim + rot_dim) or q.stride(1) != 1 or down.shape != (n, row) or down.stride(1) != 1 or \
-            q.dtype != down.dtype or cache.dtype != q.dtype or cache.dim() != 2 or cache.shape[1] % row or not cache.is_contiguous() or \
+    if (q is not None and (q.shape != (n, heads * (head_dim + rot_dim)) or q.stride(1) != 1 or q.dtype != down.dtype)) or \
+            down.shape[1] != row or down.stride(1) != 1 or \
+            cache.dtype != down.dtype or cache.dim() != 2 or cache.shape[1] % row or not cache.is_contiguous() or \
             weight.numel() != rank or weight.dtype != torch.float32 or freqs.dtype != torch.float32 or 2 * freqs.numel() > rot_dim:
         raise KernelError("latent_prepare: shapes do not fit")
-    _call(library("core"), "dd_latent_prepare", _ptr(q, "q"), q.stride(0), heads, head_dim, rot_dim, _ptr(down, "down"),
+    normed = None
+    if second is not None:
+        if second.shape[0] != n or second.stride(1) != 1 or second.dtype != down.dtype or second_weight is None or \
+                second_weight.numel() != second.shape[1] or second_weight.dtype != torch.float32 or not second_weight.is_contiguous():
+            raise KernelError("latent_prepare: the second latent does not fit its weight")
+        normed = torch.empty(second.shape, dtype=second.dtype, device=second.device)
+    _call(library("core"), "dd_latent_prepare", _ptr(q, "q"), 0 if q is None else q.stride(0), 0 if q is None else heads, head_dim,
+          rot_dim, _ptr(down, "down"),
           down.stride(0), rank, _ptr(weight), float(eps), _ptr(freqs), freqs.numel(), _ptr(token_entry, "token_entry", torch.int32),
           _ptr(positions, "positions", torch.int32), _ptr(block_table, "block_table", torch.int32), block_table.shape[1],
-          _ptr(cache), cache.shape[0], cache.shape[1] // row, n, _dt(q.dtype), _ptr(error_flag(q.device)), _stream())
+          _ptr(cache), cache.shape[0], cache.shape[1] // row, n, _dt(down.dtype), _ptr(error_flag(down.device)), _stream(),
+          1 if interleaved else 0, _ptr(second, "second"), 0 if second is None else second.stride(0),
+          0 if second is None else second.shape[1], _ptr(second_weight, "second_weight"), _ptr(normed), 0 if normed is None else normed.stride(0))
+    return normed
 
 
-def per_head_linear(x, w, in_head, out_head=None, tail=0, out=None, kernel=None):
+def per_head_linear(x, w, in_head, out_head=None, tail=0, out=None, kernel=None, turn=None):
     """out[t, h, :J] = w[h] @ x[t, h, :I], out[t, h, J:J+tail] = x[t, h, I:I+tail]: every head's piece of a row times the
     head's own matrix. x: a row view whose head h starts at h * in_head; w: [heads, J, I] contiguous, x's type; out: rows
     whose head h starts at h * out_head (default J + tail, packed). float32 sums in an order that does not depend on the
-    batch. kernel: 'mma' (bfloat16 on the tensor cores, tiles of 64 tokens x 128 outputs), 'plain', or None for 'mma'
+    batch. turn = (freqs, positions, interleaved): the first 2 * len(freqs) elements of the tail are rotated by position *
+    freqs as they are copied. kernel: 'mma' (bfloat16 on the tensor cores, tiles of 64 tokens x 128 outputs), 'plain', or None for 'mma'
     where the sizes allow it."""
     heads, J, I = w.shape
     out_head = J + tail if out_head is None else out_head
     n = x.shape[0]
     if x.stride(1) != 1 or w.dtype != x.dtype or not w.is_contiguous() or x.shape[1] < (heads - 1) * in_head + I + tail:
         raise KernelError("per_head_linear: shapes do not fit")
+    turned = (None, 0, 1, None)
+    if turn is not None:
+        freqs, positions, interleaved = turn
+        if freqs.dtype != torch.float32 or 2 * freqs.numel() > tail or positions.numel() != n:
+            raise KernelError("per_head_linear: the rotation does not fit the tail")
+        turned = (_ptr(freqs, "freqs"), freqs.numel(), 1 if interleaved else 0, _ptr(positions, "positions", torch.int32))
     if out is None:
         out = torch.empty((n, heads * out_head), dtype=x.dtype, device=x.device)
     if kernel is None:
@@ -692,10 +719,10 @@ def per_head_linear(x, w, in_head, out_head=None, tail=0, out=None, kernel=None)
             x.stride(0), int(in_head), out.stride(0), int(out_head), I, BF16)) else "plain"
     if kernel == "mma":
         _call(library("tensor"), "dd_per_head_mma", _ptr(x, "x"), x.stride(0), int(in_head), _ptr(w, "w"), _ptr(out, "out"),
-              out.stride(0), int(out_head), n, heads, I, J, int(tail), _stream())
+              out.stride(0), int(out_head), n, heads, I, J, int(tail), _stream(), *turned)
         return out
     _call(library("core"), "dd_per_head_linear", _ptr(x, "x"), x.stride(0), int(in_head), _ptr(w, "w"), _ptr(out, "out"),
-          out.stride(0), int(out_head), n, heads, I, J, int(tail), _dt(x.dtype), _stream())
+          out.stride(0), int(out_head), n, heads, I, J, int(tail), _dt(x.dtype), _stream(), *turned)
     return out
 
 
@@ -713,12 +740,14 @@ def attention_latent_splits(n_tokens, n_entries, n_heads, context, device):
     return max(1, min(-(-2 * sm_count(device) // tiles), -(-context // 64), 32))
 
 
-def attention_latent(q, cache, entry_start, entry_pos0, block_table, n_heads, v_dim, scale, n_splits=1, sink=None, out=None):
+def attention_latent(q, cache, entry_start, entry_pos0, block_table, n_heads, v_dim, scale, n_splits=1, sink=None, out=None,
+                     window=None, gate=None):
     """Tensor-core causal attention of runs of consecutive tokens over cached latent rows: the cache
     ([pages, page_size * row] bfloat16) holds one row a token, which is every head's key, and whose first v_dim elements
     are the value. q: [N, n_heads * row] row view; entry_start int32 [E+1], entry_pos0 int32 [E]; block_table row e is
     entry e's pages. sink: float32 [n_heads], exp(sink) joins the softmax's denominator. n_splits: into how many pieces
-    a row's keys are cut (partial sums merged by a second kernel). Returns [N, n_heads * v_dim]. The softmax weights meet
+    a row's keys are cut (partial sums merged by a second kernel). window: a token sees itself and the window - 1 keys
+    before it. gate: [N, n_heads] row view, a head's result is multiplied by its logistic function. Returns [N, n_heads * v_dim]. The softmax weights meet
     the values as two bfloat16 terms. See attention_latent_supported for the sizes."""
     n, n_entries = q.shape[0], entry_pos0.numel()
     row = q.shape[1] // n_heads
@@ -727,6 +756,7 @@ def attention_latent(q, cache, entry_start, entry_pos0, block_table, n_heads, v_
         raise KernelError("attention_latent: q or the entry arrays do not fit the cache")
     if sink is not None and (sink.numel() != n_heads or sink.dtype != torch.float32 or not sink.is_contiguous()):
         raise KernelError("attention: the sink must be float32 [heads]")
+    _, gate_ptr, gate_stride = _gate_args(gate, q, n_heads, None)
     if out is None:
         out = torch.empty((n, n_heads * v_dim), dtype=q.dtype, device=q.device)
     part_o = part_ml = None
@@ -737,7 +767,93 @@ def attention_latent(q, cache, entry_start, entry_pos0, block_table, n_heads, v_
           _ptr(entry_start, "entry_start", torch.int32), _ptr(entry_pos0, "entry_pos0", torch.int32), n_entries, n,
           _ptr(block_table, "block_table", torch.int32), block_table.shape[1], _ptr(out, "out"), out.stride(0),
           _ptr(part_o), _ptr(part_ml), n_heads, row, int(v_dim), cache.shape[1] // row, cache.shape[0], float(scale),
-          int(n_splits), _ptr(error_flag(q.device)), _ptr(sink, "sink"), _stream(), n_kernels=2 if n_splits > 1 else 1)
+          int(n_splits), _ptr(error_flag(q.device)), _ptr(sink, "sink"), _stream(), 0 if window is None else int(window), gate_ptr,
+          gate_stride, n_kernels=2 if n_splits > 1 else 1)
+    return out
+
+
+def token_mix(x, weight, eps, out_dtype, offset=0.0, keep=True, weight2=None, mu=None, state=None, token_entry=None, entry_start=None,
+              entry_slot=None, rows_per_mix=None):
+    """One pass over float32 rows x [N, width]: (n, n2, mixes) with n = x / sqrt(mean(x^2) + eps) * (offset + weight) (None with
+    keep False), n2 the same with weight2 (None without one), and, with mu float32 [S, width], mixes [S, rows_per_mix or N,
+    width], mixes[s][t] = n[t] + (n[t-1] - n[t]) * mu[s] in its first N rows (the others are not written); n[t-1] of an
+    entry's first token is the float32 row of ``state`` [slots, width], which then becomes the entry's last normed row.
+    float32 inside, rounded once to out_dtype."""
+    _rows(x, "x")
+    n, width = x.shape
+    if not x.is_contiguous() or x.dtype != torch.float32:
+        raise KernelError("token_mix input must be contiguous float32")
+    for v in (weight, weight2):
+        if v is not None and (v.numel() != width or v.dtype != torch.float32 or not v.is_contiguous()):
+            raise KernelError("token_mix: a weight must be float32 [width]")
+    empty = lambda *shape: torch.empty(shape, dtype=out_dtype, device=x.device)
+    count, planes, mixes = 0, n, None
+    if mu is not None:
+        count, planes = mu.shape[0], int(rows_per_mix or n)
+        if mu.shape[1] != width or mu.dtype != torch.float32 or not mu.is_contiguous() or state is None or planes < n or \
+                state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (width,):
+            raise KernelError("token_mix: the blends' weights or the state do not fit")
+        mixes = empty(count, planes, width)
+    out1 = empty(n, width) if keep else None
+    out2 = empty(n, width) if weight2 is not None else None
+    _call(library("core"), "dd_token_mix", _ptr(x, "x"), _ptr(weight), _ptr(weight2), _ptr(mu), count, _ptr(state),
+          _ptr(token_entry, "token_entry", torch.int32), _ptr(entry_start, "entry_start", torch.int32),
+          _ptr(entry_slot, "entry_slot", torch.int32), _ptr(out1), _ptr(out2), _ptr(mixes), planes * width, n, width, float(eps),
+          float(offset), _dt(out_dtype), _stream())
+    return out1, out2, mixes
+
+
+def _time_operands(r, k, v, decay_in, w0, u, heads, head_dim, value_dim, *more):
+    n = r.shape[0]
+    qk, vw = heads * head_dim, heads * value_dim
+    if r.shape != (n, qk) or k.shape != r.shape or v.shape != (n, vw) or decay_in.shape != (n, qk) or decay_in.dtype != torch.float32 or \
+            not decay_in.is_contiguous() or any(t.stride(0) != r.stride(0) or t.stride(1) != 1 or t.dtype != r.dtype for t in (r, k, v, *more)) or \
+            any(p.numel() != qk or p.dtype != torch.float32 or not p.is_contiguous() for p in (w0, u)):
+        raise KernelError("time mixing: the operands do not fit the heads (row views of one stride and type, float32 parameters)")
+    return n, qk, vw
+
+
+def time_prepare(r, k, v, decay_in, w0, u, heads, head_dim, value_dim):
+    """The recurrence's operands of a step as float32 rows: (r, k [N, heads*head_dim], v [N, heads*value_dim], fade = 1 -
+    exp(-exp(decay_in + w0)) [N, heads*head_dim], bonus = sum over a head of r * u * k [N, heads]). r, k, v: row views of one
+    stride; decay_in float32 [N, heads*head_dim]; w0, u float32 [heads*head_dim]."""
+    n, qk, vw = _time_operands(r, k, v, decay_in, w0, u, heads, head_dim, value_dim)
+    f32 = lambda w: torch.empty((n, w), dtype=torch.float32, device=r.device)
+    ro, ko, vo, fade, bonus = f32(qk), f32(qk), f32(vw), f32(qk), f32(heads)
+    _call(library("core"), "dd_time_prepare", _ptr(r, "r"), _ptr(k, "k"), _ptr(v, "v"), r.stride(0), _ptr(decay_in), _ptr(w0), _ptr(u),
+          _ptr(ro), _ptr(ko), _ptr(vo), _ptr(fade), _ptr(bonus), n, heads, head_dim, value_dim, _dt(r.dtype), _stream())
+    return ro, ko, vo, fade, bonus
+
+
+def time_scan(r, k, v, fade, bonus, entry_start, entry_slot, state, heads, head_dim, value_dim, out=None):
+    """The recurrence of a step: per entry and head, from the state in row entry_slot[e] of ``state`` (float32 [slots,
+    *delta_state_shape(...)], read and written), token by token: o = S^T r + bonus * v; S = S - fade[:, None] * S + k v^T.
+    Operands as ``time_prepare`` leaves them. Returns o float32 [N, heads*value_dim]."""
+    n = r.shape[0]
+    ok = all(t.dtype == torch.float32 and t.is_contiguous() for t in (r, k, v, fade, bonus, state))
+    if not ok or r.shape != (n, heads * head_dim) or k.shape != r.shape or fade.shape != r.shape or v.shape != (n, heads * value_dim) or \
+            bonus.shape != (n, heads) or tuple(state.shape[1:]) != delta_state_shape(heads, head_dim, value_dim):
+        raise KernelError("time_scan: shapes do not fit the state")
+    if out is None:
+        out = torch.empty((n, heads * value_dim), dtype=torch.float32, device=r.device)
+    _call(library("core"), "dd_time_scan", _ptr(r), _ptr(k), _ptr(v), _ptr(fade), _ptr(bonus),
+          _ptr(entry_start, "entry_start", torch.int32), _ptr(entry_slot, "entry_slot", torch.int32), entry_slot.numel(), _ptr(state),
+          _ptr(out), heads, head_dim, value_dim, _stream())
+    return out
+
+
+def time_step(r, k, v, gate, decay_in, w0, u, weight, eps, entry_slot, state, heads, head_dim, value_dim, out=None):
+    """A step of single tokens (row e is entry e) in one kernel: ``time_prepare``, ``time_scan`` and ``retention_finish`` with
+    its weight. r, k, v, gate: row views of one stride; weight float32 [heads*value_dim]. Returns [N, heads*value_dim] in r's type."""
+    n, qk, vw = _time_operands(r, k, v, decay_in, w0, u, heads, head_dim, value_dim, gate)
+    if gate.shape != (n, vw) or weight.numel() != vw or weight.dtype != torch.float32 or entry_slot.numel() != n or \
+            state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != delta_state_shape(heads, head_dim, value_dim):
+        raise KernelError("time_step: shapes do not fit the state")
+    if out is None:
+        out = torch.empty((n, vw), dtype=r.dtype, device=r.device)
+    _call(library("core"), "dd_time_step", _ptr(r, "r"), _ptr(k, "k"), _ptr(v, "v"), _ptr(gate, "gate"), r.stride(0), _ptr(decay_in), _ptr(w0),
+          _ptr(u), _ptr(weight), float(eps), _ptr(entry_slot, "entry_slot", torch.int32), n, _ptr(state), _ptr(out), out.stride(0), heads,
+          head_dim, value_dim, _dt(r.dtype), _stream())
     return out
 
 
@@ -813,16 +929,18 @@ def retention(q, k, v, positions, entry_start, entry_slot, decay, key_scale, sta
     return out
 
 
-def retention_finish(o, gate, heads, eps, out_dtype, out=None):
-    """out[t, head] = o[t, head] / sqrt(mean(o[t, head]^2) + eps) * silu(gate[t, head]); o float32 [N, heads*dv], gate a
-    row view [N, heads*dv] in out_dtype."""
+def retention_finish(o, gate, heads, eps, out_dtype, out=None, weight=None):
+    """out[t, head] = o[t, head] / sqrt(mean(o[t, head]^2) + eps) (* weight[head]) * silu(gate[t, head]); o float32 [N,
+    heads*dv], gate a row view [N, heads*dv] in out_dtype, weight float32 [heads*dv] or None."""
     n, total = o.shape
+    if weight is not None and (weight.numel() != total or weight.dtype != torch.float32 or not weight.is_contiguous()):
+        raise KernelError("retention_finish: the weight must be float32 [heads * value_dim]")
     if gate.shape != (n, total) or gate.stride(1) != 1 or gate.dtype != out_dtype or not o.is_contiguous() or total % heads:
         raise KernelError("retention_finish: the gate does not fit the read-out")
     if out is None:
         out = torch.empty((n, total), dtype=out_dtype, device=o.device)
     _call(library("core"), "dd_retention_finish", _ptr(o, "o", torch.float32), _ptr(gate, "gate"), gate.stride(0), _ptr(out, "out"),
-          out.stride(0), n, heads, total // heads, float(eps), _dt(out_dtype), _stream())
+          out.stride(0), n, heads, total // heads, float(eps), _dt(out_dtype), _stream(), _ptr(weight))
     return out
 
 
@@ -921,9 +1039,11 @@ def grouped_rows(n_tokens, top, n_experts, tile):
     return -(-(pairs + min(n_experts, pairs) * (tile - 1)) // tile) * tile
 
 
-def route_by_table(ids, table, n_experts, tile):
+def route_by_table(ids, table, n_experts, tile, n_identity=0):
     """ids int32 [N], table int32 [vocab, K] -> (pair_row [N*K], row_token [rows], tile_group [rows/tile]). ids None:
-    token t reads row t of the table (the step's own choices, [N, K], as ``route_by_score`` leaves them)."""
+    token t reads row t of the table (the step's own choices, [N, K], as ``route_by_score`` leaves them). Table entries
+    n_experts .. n_experts + n_identity - 1 are experts whose output is the token's own input: they get no rows, their pairs
+    the pair_row -2 (see ``combine_rows``)."""
     vocab, top = table.shape
     n = vocab if ids is None else ids.numel()
     rows = grouped_rows(n, top, n_experts, tile)
@@ -931,27 +1051,33 @@ def route_by_table(ids, table, n_experts, tile):
     row_token = torch.empty((rows,), dtype=torch.int32, device=table.device)
     tile_group = torch.empty((rows // tile,), dtype=torch.int32, device=table.device)
     _call(library("core"), "dd_route_by_table", _ptr(ids, "ids", torch.int32), _ptr(table, "table", torch.int32), n, vocab, top,
-          n_experts, tile, rows, _ptr(pair_row), _ptr(row_token), _ptr(tile_group), _ptr(error_flag(table.device)), _stream())
+          n_experts, tile, rows, _ptr(pair_row), _ptr(row_token), _ptr(tile_group), _ptr(error_flag(table.device)), _stream(),
+          int(n_identity))
     return pair_row, row_token, tile_group
 
 
-def route_by_score(y, router, n_experts, top, groups=1, keep=1, weight_scale=1.0, shared_gate=False):
+def route_by_score(y, router, n_experts, top, groups=1, keep=1, weight_scale=1.0, shared_gate=False, softmax=False,
+                   correction=None, renormalize=False):
     """Normed rows y [N, width] and the router's matrix [n_experts (+ 1), width] (one storage type) -> (chosen int32
     [N, top], pair_weight float32 [N, top], shared_scale float32 [N] or None). logit = y . router row as float32 sums of
     exact products, score = sigmoid(logit); the experts form ``groups`` equal runs of neighbours, a run's worth is the sum
     of its two largest scores, only the ``keep`` worthiest runs stay eligible; the ``top`` largest eligible scores win, each
     weighing score * weight_scale. shared_gate: the router's last row is a shared unit's gate vector, whose sigmoid is
-    returned as shared_scale."""
+    returned as shared_scale. softmax: the scores are the softmax of the n_experts logits instead. correction: float32
+    [n_experts], added to the scores for the choice only. renormalize: the chosen weights are divided by the chosen scores'
+    sum + 1e-20."""
     _rows(y, "y"), _rows(router, "router")
     n, width = y.shape
     if router.shape != (n_experts + (1 if shared_gate else 0), width) or router.dtype != y.dtype:
         raise KernelError(f"route_by_score: router {tuple(router.shape)} {router.dtype} does not fit {n_experts} experts over y {tuple(y.shape)} {y.dtype}")
+    if correction is not None and (correction.numel() != n_experts or correction.dtype != torch.float32 or not correction.is_contiguous()):
+        raise KernelError("route_by_score: the correction must be float32 [experts]")
     chosen = torch.empty((n, top), dtype=torch.int32, device=y.device)
     weight = torch.empty((n, top), dtype=torch.float32, device=y.device)
     shared = torch.empty((n,), dtype=torch.float32, device=y.device) if shared_gate else None
     _call(library("core"), "dd_route_by_score", _ptr(y, "y"), y.stride(0), _ptr(router, "router"), router.stride(0), width, n,
           n_experts, top, groups, keep, float(weight_scale), n_experts if shared_gate else -1, _ptr(chosen), _ptr(weight),
-          _ptr(shared), _dt(y.dtype), _stream())
+          _ptr(shared), _dt(y.dtype), _stream(), 1 if softmax else 0, _ptr(correction), 1 if renormalize else 0)
     return chosen, weight, shared
 
 
@@ -1025,16 +1151,20 @@ def gated_unit(gate_up, limit, alpha, out=None, form="clamped_swish", row_scale=
     return out
 
 
-def combine_rows(y, pair_row, stream_rows, top, weight, pair_weight=None):
+def combine_rows(y, pair_row, stream_rows, top, weight, pair_weight=None, own=None):
     """stream_rows[t] += weight * sum over k of (pair_weight[t*top + k] *) y[pair_row[t*top + k]] (float32, k ascending),
-    in place. pair_weight: float32 [N * top] or None."""
+    in place. pair_weight: float32 [N * top] or None. own: [N, width] contiguous rows; where pair_row is -2, own[t] stands in
+    for a row of y."""
     if y.dtype != torch.float32 or stream_rows.dtype != torch.float32 or not y.is_contiguous() or not stream_rows.is_contiguous():
         raise KernelError("combine_rows: float32 contiguous rows wanted")
     if pair_weight is not None and (pair_weight.numel() != stream_rows.shape[0] * top or pair_weight.dtype != torch.float32
                                     or not pair_weight.is_contiguous()):
         raise KernelError("combine_rows: pair_weight must be float32 [tokens * top]")
+    if own is not None and (own.shape != stream_rows.shape or not own.is_contiguous()):
+        raise KernelError("combine_rows: own must hold a contiguous row per token")
     _call(library("core"), "dd_combine_rows", _ptr(y), _ptr(pair_row, "pair_row", torch.int32), _ptr(stream_rows),
-          stream_rows.shape[0], stream_rows.shape[1], int(top), float(weight), _stream(), _ptr(pair_weight, "pair_weight"))
+          stream_rows.shape[0], stream_rows.shape[1], int(top), float(weight), _stream(), _ptr(pair_weight, "pair_weight"),
+          _ptr(own, "own"), F32 if own is None else _dt(own.dtype))
     return stream_rows
 
 

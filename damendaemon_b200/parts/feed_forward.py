@@ -163,7 +163,8 @@ class ScoreRoutedExperts(FeedForward):
     unit's gate.
     From there on the step is that of experts chosen by a table: the (token, choice) pairs sorted by expert on the
     device, the normed rows gathered in that order, two grouped products (on the tensor cores the first with the gated
-    unit in its epilogue), and each token's rows added, weighted, in the order of its choices, into the float32 stream.
+    unit in its epilogue), and each token's rows added, weighted, in the order of its choices, into the float32 stream
+    (an identity expert's output is the token's own normed row: it has no row in the grouped products).
     The shared unit's gate multiplies its hidden row before the down product, whose epilogue adds into the stream.
     Launch shapes depend on the step's counts only, so a step can be replayed from a graph."""
     graph_safe = True
@@ -175,15 +176,16 @@ class ScoreRoutedExperts(FeedForward):
             _check_unit(u)
         if any((u.inner, u.limit, u.alpha, u.activation) != (first.inner, first.limit, first.alpha, first.activation) for u in spec.experts):
             raise ValueError("the experts of one layer must have one size and one form")
-        E = len(spec.experts)
-        if not 0 < spec.top <= E or spec.groups <= 0 or E % spec.groups or not 0 < spec.keep_groups <= spec.groups or \
+        E = self.outputs = len(spec.experts) + spec.identity
+        if spec.identity < 0 or not 0 < spec.top <= E or spec.groups <= 0 or E % spec.groups or not 0 < spec.keep_groups <= spec.groups or \
                 spec.top > E // spec.groups * spec.keep_groups:
             raise ValueError(f"{spec.top} experts per token of {E} in {spec.groups} groups of which {spec.keep_groups} stay")
-        if spec.score != "sigmoid":
-            raise ValueError(f"router score {spec.score!r} is not supported; known: ['sigmoid']")
+        if spec.score not in ("sigmoid", "softmax"):
+            raise ValueError(f"router score {spec.score!r} is not supported; known: ['sigmoid', 'softmax']")
         if spec.shared_gate and spec.shared is None:
             raise ValueError("a shared unit's gate without a shared unit")
         self.router = weights[self._router_key(spec)]
+        self.correction = weights[spec.correction] if spec.correction else None
         self.tensor_cores = grouped_on_tensor_cores(runtime, runtime.dtype, spec.width, first.inner)
         self.gate_up = torch.stack([torch.cat([weights[u.gate_weight], weights[u.up_weight]], dim=0) for u in spec.experts])
         self.down = torch.stack([weights[u.down_weight] for u in spec.experts])
@@ -205,12 +207,14 @@ class ScoreRoutedExperts(FeedForward):
 
     @staticmethod
     def tensor_decls(spec):
-        E = len(spec.experts)
+        E = len(spec.experts) + spec.identity
         if spec.shared_gate:
             decls = [TensorDecl(spec.router + "+" + spec.shared_gate, (E + 1, spec.width), "matrix", False,
                                 ((spec.router, (E, spec.width)), (spec.shared_gate, (1, spec.width))))]
         else:
             decls = [TensorDecl(spec.router, (E, spec.width), "matrix")]
+        if spec.correction:
+            decls.append(TensorDecl(spec.correction, (E,), "vector"))
         for unit in spec.experts:
             decls += _unit_decls(unit, spec.width)
         if spec.shared is not None:
@@ -221,15 +225,17 @@ class ScoreRoutedExperts(FeedForward):
         s, rt = self.spec, self.runtime
         unit, E = s.experts[0], len(s.experts)
         # the router's logits (float32 sums of exact products, whatever the storage type) and the choice, in one kernel
-        chosen, pair_weight, shared_gate = kernels.route_by_score(y, self.router, E, s.top, s.groups, s.keep_groups, s.weight_scale,
-                                                                  shared_gate=bool(s.shared_gate))
+        chosen, pair_weight, shared_gate = kernels.route_by_score(y, self.router, self.outputs, s.top, s.groups, s.keep_groups,
+                                                                  s.weight_scale, shared_gate=bool(s.shared_gate),
+                                                                  softmax=s.score == "softmax", correction=self.correction,
+                                                                  renormalize=s.renormalize)
         if self.shared is not None:
             hidden = kernels.gated_unit(linear(rt, y, self.shared[0]), s.shared.limit, s.shared.alpha, form=s.shared.activation,
                                         row_scale=shared_gate)
             residual = linear(rt, hidden, self.shared[1], residual=residual, out_dtype=residual.dtype, out=residual)
         tile = grouped_tile(self.tensor_cores, y.shape[0] * s.top, E)
-        pair_row, row_token, tile_group = kernels.route_by_table(None, chosen, E, tile)
+        pair_row, row_token, tile_group = kernels.route_by_table(None, chosen, E, tile, n_identity=s.identity)
         rows = kernels.gather_rows(y, row_token)
         hidden = grouped_gated_unit(self.tensor_cores, rows, self.gate_up, tile_group, tile, unit.limit, unit.alpha, unit.activation)
         out = grouped_linear(self.tensor_cores, hidden, self.down, tile_group, tile, out_dtype=torch.float32)
-        return kernels.combine_rows(out, pair_row, residual, s.top, 1.0, pair_weight=pair_weight.view(-1))
+        return kernels.combine_rows(out, pair_row, residual, s.top, 1.0, pair_weight=pair_weight.view(-1), own=y if s.identity else None)

@@ -2,7 +2,8 @@
 
 'linear': the final norm on the wanted rows only, then logits = y . W^T (+ bias); W may be the embedding's
 table (damendaemon/gpt2.py:18,65-66: ``head is embed``, the norm after the last prompt row was picked); with ``softcap`` c
-the logits become c * tanh(logits / c).
+the logits become c * tanh(logits / c). A scale of the logits is folded into the
+weights of the head's own norm (and into the bias), so it costs no pass over the logits.
 """
 from __future__ import annotations
 
@@ -22,6 +23,9 @@ class LinearHead(Head):
         self.norm = lookup(NORMS, spec.norm, "norm")(spec.norm, weights, runtime)
         self.weight = weights[spec.weight]
         self.bias = weights[spec.bias] if spec.bias else None
+        if spec.scale != 1.0:
+            self.norm.scale_output(spec.scale)
+            self.bias = None if self.bias is None else self.bias * spec.scale
 
     @staticmethod
     def tensor_decls(spec):

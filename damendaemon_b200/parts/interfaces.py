@@ -14,7 +14,8 @@
 
 Embedding         tensor_decls(spec); forward(ctx, position) -> float32 residual stream [N,width]
 Head              tensor_decls(spec); forward(x, ctx) -> float32 logits [ctx.n_wanted, vocab] at rows ctx.want_rows
-Norm              tensor_decls(spec); forward(x_f32 [N,width], row_index=None) -> [N,width] engine dtype
+Norm              tensor_decls(spec); forward(x_f32 [N,width], row_index=None) -> [N,width] engine dtype;
+                  scale_output(factor): everything it returns is multiplied by factor from then on
 PositionEncoding  tensor_decls(spec); embedding_table() -> table or None (added to the token
                   embedding by the fused embedding kernel); on_embedding(x, ctx) -> x for
                   encodings that act there without a table; on_query_key(q, k, ctx) -> (q, k)
@@ -22,7 +23,10 @@ PositionEncoding  tensor_decls(spec); embedding_table() -> table or None (added 
 Mixer             tensor_decls(spec); cache_needs(spec) -> [a paged need (cache/manager.py: PagedKeyValues, or any
                   PagedNeed of the mixer's own) | RequestState]; forward(y, residual, ctx, cache, position) ->
                   residual + mix(y)   (float32 [N,width]); optionally portion_multiple: where the mixer likes a
-                  prompt to be cut (the engine passes the largest one on to the scheduler)
+                  prompt to be cut (the engine passes the largest one on to the scheduler). A mixer that reads
+                  blends of its input with the token before (mix_weights [S, width], a state named 'shift') may
+                  offer forward_mixes(mixes [S, >= N, width], residual, ctx, cache, position) and
+                  mix_rows(n_tokens) (rows it wants a blend padded to): the arrangement then has the norm make them
 FeedForward       tensor_decls(spec); forward(y, residual, ctx) -> residual + ff(y)
 Arrangement       cls(layer_spec, norms, mixer, feed_forward), norms being the built norms of layer_spec.norms in
                   order; forward(x, ctx, cache, position) -> x

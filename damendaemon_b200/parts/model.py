@@ -5,7 +5,7 @@ import torch
 
 from .. import kernels
 from . import (attention, block, delta_rule, embedding, feed_forward, head, latent_attention, linear_recurrence, norms,  # noqa: F401
-               positions, retention, side_by_side, state_space)  # noqa: F401  (register the built-in parts)
+               positions, retention, side_by_side, state_space, time_mix)  # noqa: F401  (register the built-in parts)
 from .spec import TensorDecl
 from .registry import ARRANGEMENTS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSITIONS, lookup
 

@@ -27,6 +27,10 @@ class LayerNorm(Norm):
     def forward(self, x, row_index=None, out_dtype=None):
         return kernels.layernorm(x, self.gamma, self.beta, self.spec.eps, out_dtype or self.runtime.dtype, row_index)
 
+    def scale_output(self, factor):
+        self.gamma = self.gamma * factor
+        self.beta = None if self.beta is None else self.beta * factor
+
 
 @register_norm("rmsnorm")
 class RmsNorm(Norm):
@@ -36,7 +40,7 @@ class RmsNorm(Norm):
         if spec.groups < 1 or spec.width % spec.groups:
             raise ValueError(f"a row of {spec.width} does not fall into {spec.groups} equal stretches")
         self.spec, self.runtime = spec, runtime
-        self.weight = weights[spec.weight]
+        self.weight, self.offset = weights[spec.weight], spec.weight_offset
 
     @staticmethod
     def tensor_decls(spec):
@@ -44,12 +48,37 @@ class RmsNorm(Norm):
 
     def forward(self, x, row_index=None, out_dtype=None):
         return kernels.rmsnorm(x, self.weight, self.spec.eps, out_dtype or self.runtime.dtype, row_index,
-                               offset=self.spec.weight_offset, groups=self.spec.groups)
+                               offset=self.offset, groups=self.spec.groups)
+
+    def scale_output(self, factor):
+        """Multiply everything the norm returns (folded into the weight, which then is the factor itself)."""
+        self.weight, self.offset = (self.offset + self.weight) * factor, 0.0
+
+    def forward_pair(self, other, x):
+        """This norm's and another RMS norm's rows of the same x, in one pass over it."""
+        y, z, _ = kernels.token_mix(x, self.weight, self.spec.eps, self.runtime.dtype, offset=self.offset, weight2=other.weight)
+        return y, z
+
+    def forward_mixes(self, x, mu, state, ctx, other=None, rows_per_mix=None):
+        """Blends of every normed row with the normed row before it (kernels.token_mix), and, of the same x, the rows of
+        ``other`` (an RMS norm with the same eps and offset, or None), in one pass: (mixes, the other norm's rows)."""
+        if self.spec.groups != 1:
+            raise ValueError("blends with the row before are made of rows normed whole, not in groups")
+        _, z, mixes = kernels.token_mix(x, self.weight, self.spec.eps, self.runtime.dtype, offset=self.offset, keep=False,
+                                        weight2=None if other is None else other.weight, mu=mu, state=state,
+                                        token_entry=ctx.token_entry, entry_start=ctx.entry_start, entry_slot=ctx.entry_slot,
+                                        rows_per_mix=rows_per_mix)
+        return mixes, z
+
+    def pairs_with(self, other):
+        """Whether one pass can compute both norms of the same row: RMS norms of one width, eps and offset, in one group."""
+        return isinstance(other, RmsNorm) and self.spec.groups == other.spec.groups == 1 and self.spec.width == other.spec.width and \
+            self.spec.eps == other.spec.eps and self.offset == other.offset
 
     def forward_shifted(self, x, shift, state, ctx):
         """The norm of every row blended with the norm of the token before it (kernels.rmsnorm_shift), one kernel."""
         return kernels.rmsnorm_shift(x, self.weight, self.spec.eps, self.runtime.dtype, shift, state, ctx.token_entry,
-                                     ctx.entry_start, ctx.entry_slot, offset=self.spec.weight_offset, groups=self.spec.groups)
+                                     ctx.entry_start, ctx.entry_slot, offset=self.offset, groups=self.spec.groups)
 
 
 @register_norm("tanh")
@@ -70,3 +99,6 @@ class TanhNorm(Norm):
 
     def forward(self, x, row_index=None, out_dtype=None):
         return kernels.tanh_norm(x, self.alpha, self.weight, self.bias, out_dtype or self.runtime.dtype, row_index)
+
+    def scale_output(self, factor):
+        self.weight, self.bias = self.weight * factor, self.bias * factor

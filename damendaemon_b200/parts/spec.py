@@ -150,7 +150,11 @@ class LatentAttentionSpec:
     [head_dim plain | rot_dim rotated]. W_down y = [rank | rot_dim]: the first part, RMS-normed with ``latent_norm``
     (eps ``norm_eps``), is the latent c; the second, rotated, is a key part all heads share. Per head the plain key is
     W_up_key c and the value W_up_value c; score = (q_plain . k_plain + q_rot . k_rot) * scale over every earlier token;
-    ``sink`` as in ``AttentionSpec``. Only c and the rotated key part are cached."""
+    ``sink`` as in ``AttentionSpec``. Only c and the rotated key part are cached.
+
+    ``query_down`` (with ``query_norm`` and ``query_rank``): the queries go through a latent of their own, q = W_q n(W_query_down
+    y), n an RMS norm with the weight ``query_norm`` and eps ``norm_eps``. ``window`` n: a token sees itself and the n - 1
+    tokens before it. ``gate_weight`` [n_heads, width]: a head's output is multiplied by sigmoid(gate . y)."""
     kind: str            # 'latent_attention'
     width: int
     n_heads: int
@@ -168,6 +172,38 @@ class LatentAttentionSpec:
     up_value_weight: str
     out_weight: str
     sink: Optional[str] = None
+    window: Optional[int] = None
+    gate_weight: Optional[str] = None
+    query_down: Optional[str] = None
+    query_norm: Optional[str] = None
+    query_rank: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class TimeMixSpec:
+    """Time mixing with a matrix state per head and a decay per key channel that depends on the token. With y' the mixer's
+    input of the token before (zeros for a sequence's first), each of five branches s reads its own blend
+    y + (y' - y) * ``mix_weights``[s] [width]: r, k, v = W y_s ([n_heads, head_dim]), gate = silu(W_g y_g), and
+    w = exp(-exp(W_decay_up tanh(W_decay_down y_w) + decay_bias)) per head and key channel. Per head, S [head_dim, head_dim]
+    float32 per request from zero: o = (S + diag(bonus) k v^T)^T r; S <- diag(w) S + k v^T. o is divided by its root mean
+    square per head (``norm_eps``), multiplied by ``out_norm`` [n_heads * head_dim] and the gate, and projected by W_out."""
+    kind: str            # 'time_mix'
+    width: int
+    n_heads: int
+    head_dim: int
+    decay_rank: int
+    norm_eps: float
+    mix_weights: Tuple[str, str, str, str, str]      # checkpoint names, in the order r, k, v, gate, decay
+    receptance_weight: str                           # matrices [out, in]
+    key_weight: str
+    value_weight: str
+    gate_weight: str
+    decay_down: str
+    decay_up: str
+    decay_bias: str      # [n_heads * head_dim]
+    bonus: str           # [n_heads, head_dim]
+    out_norm: str
+    out_weight: str
 
 
 @dataclass(frozen=True)
@@ -348,15 +384,17 @@ class TableRoutedExpertsSpec:
 
 @dataclass(frozen=True)
 class ScoreRoutedExpertsSpec:
-    """Experts chosen per token by a router: z = W_router y in float32, s = ``score``(z) ('sigmoid'); the experts
-    form ``groups`` equal runs of neighbours, a run's worth is the sum of its two largest scores, only experts of the
+    """Experts chosen per token by a router: z = W_router y in float32, s = ``score``(z) ('sigmoid', or 'softmax' over all
+    outputs); the experts form ``groups`` equal runs of neighbours, a run's worth is the sum of its two largest scores, only experts of the
     ``keep_groups`` worthiest runs can be chosen; the ``top`` largest eligible scores win. A chosen expert's output is
-    weighted by s * weight_scale (not renormalised). ``shared``: a unit that runs for every token; with
+    weighted by s * weight_scale, or, with ``renormalize``, by s over the sum of the chosen s (+ 1e-20). ``correction`` (a
+    checkpoint name, one number per router output) is added to the scores for the choice only. The router's last ``identity``
+    outputs are experts without tensors, whose output is y itself. ``shared``: a unit that runs for every token; with
     ``shared_gate`` (a checkpoint name, [1, width]) its output is multiplied by sigmoid(gate . y)."""
     kind: str            # 'experts_by_score'
     width: int
     top: int
-    router: str          # checkpoint name of W_router [experts, width]
+    router: str          # checkpoint name of W_router [experts + identity, width]
     experts: Tuple[GatedUnitSpec, ...]       # all of one size and activation
     groups: int = 1
     keep_groups: int = 1
@@ -364,6 +402,9 @@ class ScoreRoutedExpertsSpec:
     score: str = "sigmoid"
     shared: Optional[GatedUnitSpec] = None
     shared_gate: Optional[str] = None
+    correction: Optional[str] = None
+    renormalize: bool = False
+    identity: int = 0
 
 
 @dataclass(frozen=True)
@@ -375,7 +416,8 @@ class NoFeedForwardSpec:
 class LayerSpec:
     """A layer: a mixer, a feed-forward, as many norms as its arrangement wants, and the arrangement that wires them
     ('pre_norm' takes two norms: before the mixer, before the feed-forward; 'pre_norm_mixer' one norm and no
-    feed-forward; 'parallel' one norm whose output both the mixer and the feed-forward read; 'pre_norm_shift' is
+    feed-forward; 'parallel' one norm whose output both the mixer and the feed-forward read, or two norms of the same input,
+    the first for the mixer, the second for the feed-forward; 'pre_norm_shift' is
     'pre_norm', or 'pre_norm_mixer' with one norm, whose mixer reads its normed input blended per channel with the
     normed input of the token before: n[t] + (n[t-1] - n[t]) * ``shift_weight`` [width], n[-1] = 0)."""
     arrangement: str
@@ -396,6 +438,7 @@ class EmbeddingSpec:
     width: int
     table: str           # checkpoint name
     scale: float = 1.0   # multiplies the row
+    norm: object = None  # a norm spec: the stream starts as the normed row
 
 
 @dataclass(frozen=True)
@@ -423,6 +466,7 @@ class HeadSpec:
     tied: bool = False   # W is the embedding's table (declared there, not again)
     bias: Optional[str] = None
     softcap: Optional[float] = None   # c: logits become c * tanh(logits / c)
+    scale: float = 1.0                # multiplies the logits (before the cap)
 
 
 @dataclass(frozen=True)
