@@ -374,6 +374,16 @@ TETITAR_KERNEL_PAIRS = [     # (a kernel of Tetitar, the like kernel of the clos
     ("sigmoidgate_m2048", "gatedact_m2048"), ("sigmoidgate_m8", "gatedact_m8"), ("pairnorm_m2048", "rmsnorm_m2048"), ("pairnorm_m8", "rmsnorm_m8"),
     ("embedpairs_m2048", None), ("embedpairs_m8", None),
 ]
+GODOTAR_KERNEL_PAIRS = [     # (a kernel of Godotar, the like kernel of the closest model: Derusun, for the experts Zokanex) at width 1600, 25 heads of 64
+    ("tokenmix_m2048", "groupnorm_m2048"), ("tokenmix_m8", "groupnorm_m8"), ("normpair_m2048", "rmsnorm_m2048"), ("normpair_m8", "rmsnorm_m8"),
+    ("squares_m2048", "gemm_fc_m2048"), ("squares_m8", "gemm_fc_m8"), ("squares_m64", "gemm_fc_m64"), ("lowrank_m2048", None), ("lowrank_m8", None),
+    ("timeprep_p2_t1024", "deltaprep_p2_t1024"), ("timescan_p2_t1024", "delta_p2_t1024"), ("timefinish_p2_t1024", "deltafinish_p2_t1024"),
+    ("timestep_p8_t1", "delta_p8_t1"), ("timestep_p64_t1", "delta_p64_t1"),
+    ("latentwin_prefill_p2_t1024", "latent_prefill_p2_t1024"), ("latentwin_decode_b8_c768", "latent_decode_b8_c768"),
+    ("latentwin_decode_b64_c768", "latent_decode_b64_c768"), ("latentqprep_m2048", "latentprep_m2048"), ("latentqprep_m8", "latentprep_m8"),
+    ("perheadturn_m2048", "perhead_m2048"), ("perheadturn_m8", "perhead_m8"),
+    ("grouped_softmax_m2048", "grouped_score_m2048"), ("grouped_softmax_m8", "grouped_score_m8"),
+]
 CUDA_CORE_FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12      # nominal: 148 SMs x 128 lanes x one fused multiply-add a cycle at 1,965 MHz
 
 
@@ -460,6 +470,34 @@ def tetitar_configs(size, layers, vocab=50257):
     return out
 
 
+def godotar_configs(size, layers, vocab=50257):
+    """Derusun (layers of the gated delta rule; of attention over latent rows), Zokanex (its mix with experts) and Godotar models
+    whose layers have one size: layers of time mixing and of windowed latent attention, each with the silu gated unit; and, with
+    experts (as many of them as Zokanex's, and four identity outputs), a dense layer of time mixing, then one of time mixing and
+    one of latent attention that run twice, then one of time mixing (four layers, six runs)."""
+    z = DESIGN_SIZES[size]
+    out = {k: v for k, v in derusun_configs(size, layers, vocab).items() if k in ("derusun_delta_dense", "derusun_latent_dense")}
+    out["zokanex_mixed_experts"] = zokanex_configs(size, layers, vocab)["zokanex_mixed_experts"]
+    heads = z["heads"]
+    wkv = {"heads": heads, "dim": 64, "decay_rank": 64}
+    latent = {"heads": heads, "dim": 64, "rot_dim": 64, "vdim": 64, "kv_rank": 256, "q_rank": 512, "scale": 128 ** -0.5,
+              "rot": {"dims": 64, "base": 10000.0}, "mask": {"size": 1024}}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"], "identity": 4}, "expert": {"ff": z["expert_ff"], "limit": 7.0}}
+
+    def model(entries, loop=None):
+        config = {"architecture": "Godotar", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+                  "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in entries]}
+        if loop:
+            config["loop"] = dict(zip(("start", "stop", "times"), loop))
+        return config
+    out["godotar_wkv_dense"] = model([("wkv", wkv, dense)] * layers)
+    out["godotar_latent_dense"] = model([("latent_attention", latent, dense)] * layers)
+    out["godotar_looped_experts"] = model([("wkv", wkv, dense), ("wkv", wkv, moe), ("latent_attention", latent, moe), ("wkv", wkv, moe)],
+                                          loop=(1, 3, 2))
+    return out
+
+
 def design_configs(size, layers, vocab=50257):
     """GPT-2 and two Bonatar models (dense layers only; expert layers only) whose layers have one size."""
     z = DESIGN_SIZES[size]
@@ -477,7 +515,8 @@ def design_configs(size, layers, vocab=50257):
 
 def design_bench(args):
     """``--design bonatar`` (beside GPT-2), ``--design zokanex`` (beside Bonatar, the closest model), ``--design derusun`` or
-    ``--design tetitar`` (each beside Zokanex, the closest model): prefill and decode
+    ``--design tetitar`` (each beside Zokanex, the closest model), ``--design godotar`` (beside Derusun, and Zokanex for the
+    experts): prefill and decode
     throughput at equal layer sizes (random
     bfloat16 weights, a few layers), and each kernel of the new design beside the like kernel of the other, timed in a
     chain replayed from a CUDA graph over inputs that rotate through more memory than L2 holds."""
@@ -487,7 +526,7 @@ def design_bench(args):
     hbm, tflops = measured_peaks["hbm_gbs"], measured_peaks["bf16_tflops"]
     layers = args.layers or 6
     configs_of, pairs = {"zokanex": (zokanex_configs, ZOKANEX_KERNEL_PAIRS), "derusun": (derusun_configs, DERUSUN_KERNEL_PAIRS),
-                         "tetitar": (tetitar_configs, TETITAR_KERNEL_PAIRS),
+                         "tetitar": (tetitar_configs, TETITAR_KERNEL_PAIRS), "godotar": (godotar_configs, GODOTAR_KERNEL_PAIRS),
                          "bonatar": (design_configs, DESIGN_KERNEL_PAIRS)}[args.design]
     out = {"design": args.design, "layers": layers, "dtype": "bf16", "data": "synthetic", "peaks": dict(measured_peaks, source=peaks_from),
            "sizes": {}, "kernels": [],
@@ -571,7 +610,7 @@ def main():
     parser.add_argument("--case-iters", type=int, default=50)
     parser.add_argument("--case-graph", action="store_true", help="time the kernel case as launches replayed from one CUDA graph")
     parser.add_argument("--workload", choices=sorted(WORKLOADS), help="run a scheduler workload instead of the headline bench")
-    parser.add_argument("--design", choices=("bonatar", "zokanex", "derusun", "tetitar"), help="another design beside GPT-2 (zokanex: beside Bonatar; derusun and tetitar: beside Zokanex) at equal layer sizes (prefill, decode, "
+    parser.add_argument("--design", choices=("bonatar", "zokanex", "derusun", "tetitar", "godotar"), help="another design beside GPT-2 (zokanex: beside Bonatar; derusun and tetitar: beside Zokanex; godotar: beside Derusun) at equal layer sizes (prefill, decode, "
                         "kernel by kernel) instead of the headline bench")
     parser.add_argument("--parity", action="store_true", help="the float32 engine beside the bfloat16 one: on the benchmark's model "
                         "(logit differences, greedy agreement), or with --workload on that workload (the same requests in both)")

@@ -212,7 +212,7 @@ def _latent_cache(batch, context, dev, copies):
     return caches, table
 
 
-def _latent_attention_case(batch, length, dev, decode, kernel="tensor"):
+def _latent_attention_case(batch, length, dev, decode, kernel="tensor", windowed=False):
     """Attention of 25 heads over cached latent rows of 256 + 64 (one row a token is every head's key, its first 256
     elements every head's value): `batch` prompts of `length` tokens, or (decode) `batch` single tokens behind `length`
     keys each; through the tensor-core kernel or ('rows') the general one."""
@@ -233,19 +233,23 @@ def _latent_attention_case(batch, length, dev, decode, kernel="tensor"):
         splits = 1
         keys = batch * (length * (length + 1) // 2)
     sink = torch.zeros(H, device=dev)
+    if windowed:        # a window that holds the whole context (the same keys are read) and a gate per head, no sink
+        sink, more = None, dict(window=1024 * ((context + 1023) // 1024), gate=torch.randn(tokens, H, device=dev).to(torch.bfloat16))
+    else:
+        more = {}
     if kernel == "tensor":
         start = torch.arange(batch + 1, dtype=torch.int32, device=dev) * (1 if decode else length)
         pos0 = torch.full((batch,), context - 1 if decode else 0, dtype=torch.int32, device=dev)
         if decode:
             splits = K.attention_latent_splits(batch, batch, H, context, dev)
-        run = lambda i: K.attention_latent(q, caches[i % copies], start, pos0, table, H, RANK, 0.1, n_splits=splits, sink=sink)
+        run = lambda i: K.attention_latent(q, caches[i % copies], start, pos0, table, H, RANK, 0.1, n_splits=splits, sink=sink, **more)
     else:
         run = lambda i: K.attention_rows(q, caches[i % copies], ent, pos, table, H, 0.1, n_splits=splits, kv_heads=1, v_dim=RANK,
                                          sink=sink, values_in_keys=True)
     return run, {"bytes": batch * context * row * 2 + tokens * H * (row + RANK) * 2, "flops": 2 * keys * H * (row + RANK)}
 
 
-def _latent_prepare_case(rows, dev):
+def _latent_prepare_case(rows, dev, query_rank=0):
     """A step's latent rows normed, their shared key part and the queries' rotated parts rotated, the rows written into
     their pages (25 heads of 64 + 64, latent 256 + 64)."""
     row, qw = RANK + ROT, H * (D + ROT)
@@ -258,13 +262,22 @@ def _latent_prepare_case(rows, dev):
     weight = torch.ones(RANK, device=dev)
     freqs = (10000.0 ** (-torch.arange(ROT // 2, dtype=torch.float64) * 2 / ROT)).float().to(dev)
 
+    if query_rank:      # no queries yet, but the latent they will be projected from, normed beside the row
+        second = torch.ones(query_rank, device=dev)
+
+        def run(i):
+            b = bufs[i % copies]
+            K.latent_prepare(None, b[:, qw:], weight, 1e-5, freqs, ent, pos, table, caches[0], H, D, ROT, RANK, interleaved=False,
+                             second=b[:, :query_rank], second_weight=second)
+        return run, {"bytes": rows * (query_rank * 4 + row * 4), "flops": rows * 5 * (query_rank + row)}
+
     def run(i):
         b = bufs[i % copies]
         K.latent_prepare(b[:, :qw], b[:, qw:], weight, 1e-5, freqs, ent, pos, table, caches[0], H, D, ROT, RANK)
     return run, {"bytes": rows * (H * ROT * 4 + row * 4), "flops": rows * (6 * H * ROT + 5 * row)}
 
 
-def _per_head_case(rows, dev, up, kernel=None):
+def _per_head_case(rows, dev, up, kernel=None, turned=False):
     """Every head's piece of a row times the head's own matrix (25 heads): the plain queries of 64 through the transposed
     key matrices to 256 (with the rotated 64 carried along), or (up) the attended latent rows of 256 to values of 64."""
     if up:
@@ -274,7 +287,11 @@ def _per_head_case(rows, dev, up, kernel=None):
         return run, {"bytes": rows * H * (RANK + D) * 2 + w.numel() * 2, "flops": 2 * rows * H * D * RANK}
     x = torch.randn(rows, H * (D + ROT), device=dev).to(torch.bfloat16)
     w = torch.randn(H, RANK, D, device=dev).mul_(0.1).to(torch.bfloat16)
-    run = lambda i: K.per_head_linear(x, w, D + ROT, tail=ROT, kernel=kernel)
+    turn = None
+    if turned:          # the carried elements are rotated on the way
+        freqs = (10000.0 ** (-torch.arange(ROT // 2, dtype=torch.float64) * 2 / ROT)).float().to(dev)
+        turn = (freqs, torch.arange(rows, dtype=torch.int32, device=dev) % 1024, False)
+    run = lambda i: K.per_head_linear(x, w, D + ROT, tail=ROT, kernel=kernel, turn=turn)
     return run, {"bytes": rows * H * (D + ROT + RANK + ROT) * 2 + w.numel() * 2, "flops": 2 * rows * H * D * RANK}
 
 
@@ -429,6 +446,88 @@ def _row_ops_case(which, rows, dev):
     return run, {"bytes": rows * width * 8, "flops": 2 * rows * width}
 
 
+def _token_mix_case(rows, dev, pair=False):
+    """One pass over `rows` rows of the float32 stream (width 1600): five blends of the normed row with the normed row of the
+    token before (requests of 256 tokens, or single tokens) and the row under a second norm; or (pair) the two normed rows."""
+    width = H * D
+    length = 256 if rows >= 256 else 1
+    tokens, ent, start, slot = _entries(rows // length, length, dev)
+    copies = max(2, min(24, (300 << 20) // (rows * width * 4)))
+    xs = [torch.randn(rows, width, device=dev) for _ in range(copies)]
+    w1, w2, mu = torch.zeros(width, device=dev), torch.zeros(width, device=dev), torch.rand(5, width, device=dev)
+    state = torch.zeros(rows // length, width, device=dev)
+    if pair:
+        run = lambda i: K.token_mix(xs[i % copies], w1, 1e-6, torch.bfloat16, offset=1.0, weight2=w2)
+        return run, {"bytes": rows * width * 8, "flops": 5 * rows * width}
+    run = lambda i: K.token_mix(xs[i % copies], w1, 1e-6, torch.bfloat16, offset=1.0, keep=False, weight2=w2, mu=mu, state=state,
+                                token_entry=ent, entry_start=start, entry_slot=slot)
+    return run, {"bytes": rows * width * 16, "flops": 15 * rows * width}
+
+
+def _time_mix_case(entries, length, dev, which):
+    """Time mixing of `entries` requests of `length` tokens each in one step (25 heads of 64 by 64): 'scan' the recurrence over
+    the float32 state, 'prep' its operands, 'finish' the read-out's norm, weight and gate, 'step' all three of single tokens.
+    Float32 sums on the CUDA cores."""
+    tokens, ent, start, slot = _entries(entries, length, dev)
+    inner = H * D
+    copies = max(2, min(24, (300 << 20) // max(1, tokens * 4 * inner * 4 + entries * H * D * D * 4)))
+    projs = [torch.randn(4, tokens, inner, device=dev).mul_(0.5).to(torch.bfloat16) for _ in range(copies)]
+    decay_in = torch.randn(tokens, inner, device=dev)
+    w0, u, weight = torch.full((inner,), -4.0, device=dev), torch.randn(inner, device=dev), torch.ones(inner, device=dev)
+    states = [torch.zeros(entries, *K.delta_state_shape(H, D, D), device=dev) for _ in range(copies)]
+    out = torch.empty(tokens, inner, device=dev, dtype=torch.bfloat16)
+    if which == "step":
+        def run(i):
+            p = projs[i % copies]
+            K.time_step(p[0], p[1], p[2], p[3], decay_in, w0, u, weight, 1e-6, slot, states[i % copies], H, D, D, out=out)
+        return run, {"bytes": entries * H * D * D * 8 + tokens * inner * (4 * 2 + 4 + 2), "flops": 6 * tokens * H * D * D, "fp32": True}
+    if which == "prep":
+        def run(i):
+            p = projs[i % copies]
+            K.time_prepare(p[0], p[1], p[2], decay_in, w0, u, H, D, D)
+        return run, {"bytes": tokens * inner * (3 * 2 + 4 + 4 * 4), "flops": 20 * tokens * inner, "fp32": True}
+    if which == "finish":
+        o = torch.randn(tokens, inner, device=dev)
+        run = lambda i: K.retention_finish(o, projs[i % copies][3], H, 1e-6, torch.bfloat16, out=out, weight=weight)
+        return run, {"bytes": tokens * inner * 8, "flops": 10 * tokens * inner}
+    ops = [K.time_prepare(p[0], p[1], p[2], decay_in, w0, u, H, D, D) for p in projs[:min(copies, 6)]]
+    o = torch.empty(tokens, inner, device=dev)
+    run = lambda i: K.time_scan(*ops[i % len(ops)], start, slot, states[i % copies], H, D, D, out=o)
+    return run, {"bytes": entries * H * D * D * 8 + tokens * inner * 4 * 5, "flops": 6 * tokens * H * D * D, "fp32": True}
+
+
+def _square_products_case(rows, dev):
+    """The four square products (receptance, key, value, gate) of `rows` tokens, each over its own blend (width 1600): one
+    grouped launch for few tokens, a launch each for many, as the mixer does it."""
+    width, inner = 1600, H * D
+    copies = max(2, (300 << 20) // (4 * inner * width * 2))
+    weights = [torch.randn(4, inner, width, device=dev).mul_(0.02).to(torch.bfloat16) for _ in range(copies)]
+    groups = torch.arange(4, dtype=torch.int32, device=dev)
+    work = {"bytes": 4 * inner * width * 2, "flops": 8 * rows * inner * width}
+    if rows <= 128:
+        tile = next(t for t in K.GROUPED_TCGEN05_TILES if t >= rows)
+        x = torch.randn(4 * tile, width, device=dev).to(torch.bfloat16)
+        return (lambda i: K.gemm_grouped_tcgen05(x, weights[i % copies], groups, tile)), work
+    x = torch.randn(4, rows, width, device=dev).to(torch.bfloat16)
+    out = torch.empty(4, rows, inner, device=dev, dtype=torch.bfloat16)
+
+    def run(i):
+        for j in range(4):
+            K.gemm_tcgen05(x[j], weights[i % copies][j], out=out[j])
+    return run, work
+
+
+def _low_rank_case(rows, dev, rank=64):
+    """The decay's two products of `rows` tokens (1600 -> 64 with tanh in the epilogue, 64 -> 1600 into float32)."""
+    width, inner = 1600, H * D
+    copies = 16
+    x = [torch.randn(rows, width, device=dev).to(torch.bfloat16) for _ in range(copies)]
+    down, up = torch.randn(rank, width, device=dev).mul_(0.02).to(torch.bfloat16), torch.randn(inner, rank, device=dev).mul_(0.1).to(torch.bfloat16)
+    out = torch.empty(rows, inner, device=dev)
+    run = lambda i: K.gemm_tcgen05(K.gemm_tcgen05(x[i % copies], down, activation="tanh"), up, out_dtype=torch.float32, out=out)
+    return run, {"bytes": rows * (width * 2 + inner * 4) + (width + inner) * rank * 2, "flops": 2 * rows * rank * (width + inner)}
+
+
 def _gated_act_case(rows, dev):
     """The dense gated unit between its two products: rows of [gate | up] halves (2 x 6400) -> tanh-gelu(gate) * up."""
     inner = 6400
@@ -440,6 +539,9 @@ def _gated_act_case(rows, dev):
 
 
 EXPERTS, TOP, INNER = 16, 2, 1600       # sixteen experts of a quarter of the dense inner width, two per token
+
+
+IDENTITY = 4                            # of a softmax router's sixteen outputs, the last four are the input itself
 
 
 def _grouped_case(which, tokens, dev):
@@ -467,6 +569,22 @@ def _grouped_case(which, tokens, dev):
             K.gather_rows(x, rt)
             K.combine_rows(y, pr, stream, TOP, 1.0, pair_weight=weight.view(-1))
         return run, {"bytes": tokens * TOP * width * (2 + 2 + 4) + tokens * width * 10, "flops": tokens * (TOP + 2 * EXPERTS) * width}
+    if which == "softmax":
+        # the router's logits, their softmax, a corrected choice and renormalised weights (one kernel), then the same; the last
+        # outputs are the token's own row: fewer rows to gather, the sum reads the normed rows as well
+        router, correction = torch.randn(EXPERTS, width, device=dev).mul_(0.05).to(torch.bfloat16), torch.zeros(EXPERTS, device=dev)
+        stream = torch.zeros(tokens, width, device=dev)
+        real = EXPERTS - IDENTITY
+        tile = grouped_tile(True, tokens * TOP, real)
+        y = torch.zeros(K.grouped_rows(tokens, TOP, real, tile), width, device=dev)
+
+        def run(i):
+            chosen, weight, _ = K.route_by_score(x, router, EXPERTS, TOP, softmax=True, correction=correction, renormalize=True)
+            pr, rt, tg = K.route_by_table(None, chosen, real, tile, n_identity=IDENTITY)
+            K.gather_rows(x, rt)
+            K.combine_rows(y, pr, stream, TOP, 1.0, pair_weight=weight.view(-1), own=x)
+        gathered = tokens * TOP * real // EXPERTS
+        return run, {"bytes": gathered * width * (2 + 2 + 4) + tokens * width * 12, "flops": tokens * (TOP + 2 * EXPERTS) * width}
     if which == "route":
         stream = torch.zeros(tokens, width, device=dev)
         y = torch.zeros(rows.shape[0], width, device=dev)
@@ -536,7 +654,9 @@ def build(name, device="cuda:0"):
     sinks_prefillrows_.., sinks_decoderows_..: through the general kernel) | tanhnorm_m<rows> | widenorm_m<rows> |
     ssmconv_p<requests>_t<tokens> | ssmscan_p.._t.. | ssmfinish_p.._t.. | rglrugates_p.._t.. | rglruscan_p.._t.. |
     sigmoidgate_m<rows> | pairnorm_m<rows> | embedpairs_m<rows> | unitsink_prefill_p<prompts>_t<tokens> |
-    unitsink_decode_b<batch>_c<context>; attention cases take the suffix _masked (a chunked mask and a gate on every head's
+    unitsink_decode_b<batch>_c<context> | tokenmix_m<rows> | normpair_m<rows> | timescan_p<requests>_t<tokens> | timeprep_p.._t.. |
+    timefinish_p.._t.. | timestep_p<requests>_t1 | squares_m<rows> | lowrank_m<rows> | latentwin_prefill_p.._t.. |
+    latentwin_decode_b.._c.. | latentqprep_m<rows> | perheadturn_m<rows> | grouped_softmax_m<tokens>; attention cases take the suffix _masked (a chunked mask and a gate on every head's
     output)"""
     K.library("core"), K.library("tensor")
     masked = name.endswith("_masked")          # attention cases: with a chunked mask and an output gate
@@ -559,6 +679,13 @@ def build(name, device="cuda:0"):
         # unitsink_prefill_p<prompts>_t<tokens> | unitsink_decode_b<batch>_c<context>: a window and a unit term in the softmax
         a, b = name.split("_", 2)[2][1:].replace("_t", " ").replace("_c", " ").split()
         return _sinks_case(int(a), int(b), device, parts[1] == "decode", "tensor", unit_only=True)
+    if parts[0] in ("tokenmix", "normpair", "squares", "lowrank") and len(parts) == 2 and parts[1][0] == "m":
+        rows = int(parts[1][1:])
+        return _square_products_case(rows, device) if parts[0] == "squares" else _low_rank_case(rows, device) if parts[0] == "lowrank" \
+            else _token_mix_case(rows, device, pair=parts[0] == "normpair")
+    if parts[0] in ("timescan", "timeprep", "timefinish", "timestep") and "_p" in name:
+        entries, tokens = name.split("_p")[1].split("_t")
+        return _time_mix_case(int(entries), int(tokens), device, parts[0][4:])
     if name.startswith("groupnorm_m"):
         return _group_norm_shift_case(int(name[len("groupnorm_m"):]), device)
     if name.startswith("depthmix_m"):
@@ -570,6 +697,14 @@ def build(name, device="cuda:0"):
         # latent_prefill_p<prompts>_t<tokens> | latent_decode_b<batch>_c<context>; ...rows: through the general kernel
         a, b = name.split("_", 2)[2][1:].replace("_t", " ").replace("_c", " ").split()
         return _latent_attention_case(int(a), int(b), device, parts[1].startswith("decode"), "rows" if parts[1].endswith("rows") else "tensor")
+    if parts[0] == "latentwin" and parts[1] in ("prefill", "decode"):
+        # latentwin_prefill_p<prompts>_t<tokens> | latentwin_decode_b<batch>_c<context>: with a window and a gate per head
+        a, b = name.split("_", 2)[2][1:].replace("_t", " ").replace("_c", " ").split()
+        return _latent_attention_case(int(a), int(b), device, parts[1] == "decode", windowed=True)
+    if name.startswith("latentqprep_m"):
+        return _latent_prepare_case(int(name[len("latentqprep_m"):]), device, query_rank=512)
+    if name.startswith("perheadturn_m"):
+        return _per_head_case(int(name[len("perheadturn_m"):]), device, False, turned=True)
     if name.startswith("latentprep_m"):
         return _latent_prepare_case(int(name[len("latentprep_m"):]), device)
     if parts[0] in ("perhead", "perheadup", "perheadplain", "perheadupplain"):
@@ -591,7 +726,7 @@ def build(name, device="cuda:0"):
         # retention_p<requests>_t<tokens of each>: prompts; _t1: a decode step of that many requests
         entries, tokens = name.split("_p")[1].split("_t")
         return _retention_case(int(entries), int(tokens), device, finish=name.startswith("retfinish"))
-    if parts[0] == "grouped" and len(parts) == 3 and parts[1] in ("up", "upsilu", "down", "route", "score") and parts[2][0] == "m":
+    if parts[0] == "grouped" and len(parts) == 3 and parts[1] in ("up", "upsilu", "down", "route", "score", "softmax") and parts[2][0] == "m":
         return _grouped_case(parts[1], int(parts[2][1:]), device)
     if parts[0] == "gemm" and len(parts) == 3 and parts[1] in SHAPES and parts[2][0] == "m":
         return _gemm_case(parts[1], int(parts[2][1:]), device)
