@@ -16,12 +16,15 @@
 //
 //   dd_time_prepare   the operands of a step as float32 rows: r, k, v, 1 - w, and the bonus sum_i r_i u_i k_i per head
 //   dd_time_scan      the recurrence over a step's entries. Column j of o depends on column j of S only: a block owns
-//                     (entry, head, a run of columns); a column's rows are dealt out over LPC neighbouring lanes, eight
-//                     each in registers. No token's update waits for an exchange between lanes: only the read-outs are
-//                     exchanged, four tokens side by side. Tokens are staged 16 at a time by cp.async, two buffers in turn.
+//                     (entry, head, a run of columns); a column's rows are dealt out over neighbouring lanes, and a thread
+//                     holds the same few rows of several columns in registers, so that an operand it reads from shared
+//                     memory serves them all. No token's update waits for an exchange between lanes: only the read-outs
+//                     are exchanged, those of four tokens together (spread_sums). Tokens are staged 16 at a time by
+//                     cp.async, two buffers in turn.
 //   dd_time_step      a step of single tokens in one kernel: operands, recurrence, and the read-out's norm, weight and gate;
-//                     a block owns (entry, head). Update and read-out are the scan's instructions in the scan's order.
-// The state is stored column by column ([slots, heads, dv, 8 * LPC]; rows past dk stay zero).
+//                     a block owns (entry, head), a thread eight rows of a column. The state's update is the scan's, bit for
+//                     bit.
+// The state is stored column by column ([slots, heads, dv, dkp], dkp = dk rounded up to 8 times a power of two; rows past dk stay zero).
 #include "common.cuh"
 
 namespace {
@@ -283,28 +286,49 @@ __device__ __forceinline__ float time_token(float (&s)[8], const float* r, const
     return __fadd_rn(a, b);
 }
 
-constexpr int TS_THREADS = 128;
+// N sums, of which every one of a column's LPC lanes holds a part: at every exchange (O = 1, 2, 4, .. lanes apart) a lane gives
+// away half of its sums and keeps the other half while it has more than one, so that all of them together take little more
+// exchanges than one would. Returns the index of the first sum the lane is left with, in read[0].
+template <int N, int O, int LPC>
+__device__ __forceinline__ int spread_sums(float* read, int sub) {
+    if constexpr (O >= LPC) {
+        return 0;
+    } else if constexpr (N > 1) {
+        const bool up = (sub & O) != 0;
+#pragma unroll
+        for (int i = 0; i < N / 2; ++i) {
+            const float give = up ? read[i] : read[i + N / 2];
+            const float keep = up ? read[i + N / 2] : read[i];
+            read[i] = keep + __shfl_xor_sync(0xffffffffu, give, O);
+        }
+        return (up ? N / 2 : 0) + spread_sums<N / 2, O * 2, LPC>(read, sub);
+    } else {
+        read[0] += __shfl_xor_sync(0xffffffffu, read[0], O);
+        return spread_sums<1, O * 2, LPC>(read, sub);
+    }
+}
+
 constexpr int TS_TOKENS = 16;          // tokens staged together
 
-template <int LPC>
-__global__ void __launch_bounds__(TS_THREADS)
+// R rows and C columns of the state a thread (R a multiple of 4, 16-byte pieces that lie a whole sweep of the column's LPC
+// lanes apart, so that neighbouring lanes read neighbouring pieces); THREADS / LPC * C columns a block.
+template <int R, int C, int LPC, int THREADS>
+__global__ void __launch_bounds__(THREADS)
 time_scan_kernel(const float* __restrict__ r, const float* __restrict__ k, const float* __restrict__ v, const float* __restrict__ fade,
                  const float* __restrict__ bonus, const int* __restrict__ entry_start, const int* __restrict__ entry_slot,
                  float* __restrict__ state, float* __restrict__ out, int H, int dk, int dv) {
-    constexpr int DKP = 8 * LPC, COLS = TS_THREADS / LPC;
+    constexpr int DKP = R * LPC, COLS = THREADS / LPC * C, P = R / 4;
     constexpr int BUF = TS_TOKENS * (3 * DKP + COLS) + TS_TOKENS;       // floats of one buffer: r, k, fade, v, bonus
     extern __shared__ __align__(16) float staged[];
     dd_launch_dependents();
     const int e = blockIdx.z, h = blockIdx.y;
     const int col0 = blockIdx.x * COLS;
-    const int my_col = threadIdx.x / LPC, sub = threadIdx.x % LPC;
-    const int col = col0 + my_col;
-    const bool live = col < dv;
+    const int my_col = threadIdx.x / LPC * C, sub = threadIdx.x % LPC;
     const int start = entry_start[e], end = entry_start[e + 1];
     // rows past dk and columns past dv are never copied into: they stay the zeros written here, and so do the tokens past
     // an entry's last one in its last buffer (a token of zeros leaves the state as it is)
-    for (int i = threadIdx.x; i < 2 * BUF; i += TS_THREADS) staged[i] = 0.f;
-    const bool wide = dk % 4 == 0 && dv % 4 == 0;
+    for (int i = threadIdx.x; i < 2 * BUF; i += THREADS) staged[i] = 0.f;
+    const bool wide = dk % 4 == 0 && dv % 4 == 0 && COLS % 4 == 0;
     auto stage = [&](int t0, int buf) {
         const int n = min(TS_TOKENS, end - t0);
         float* br = staged + buf * BUF;
@@ -313,7 +337,7 @@ time_scan_kernel(const float* __restrict__ r, const float* __restrict__ k, const
         float* bv = bf + TS_TOKENS * DKP;
         float* bb = bv + TS_TOKENS * COLS;
         if (wide) {
-            for (int i = threadIdx.x; i < n * (DKP / 4); i += TS_THREADS) {
+            for (int i = threadIdx.x; i < n * (DKP / 4); i += THREADS) {
                 const int tt = i / (DKP / 4), c = (i % (DKP / 4)) * 4;
                 if (c < dk) {
                     const size_t at = ((size_t)(t0 + tt) * H + h) * dk + c;
@@ -322,14 +346,12 @@ time_scan_kernel(const float* __restrict__ r, const float* __restrict__ k, const
                     tm_cp_async<16>(bf + tt * DKP + c, fade + at);
                 }
             }
-            if (COLS >= 4) {
-                for (int i = threadIdx.x; i < n * (COLS / 4); i += TS_THREADS) {
-                    const int tt = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
-                    if (col0 + c < dv) tm_cp_async<16>(bv + tt * COLS + c, v + ((size_t)(t0 + tt) * H + h) * dv + col0 + c);
-                }
+            for (int i = threadIdx.x; i < n * (COLS / 4); i += THREADS) {
+                const int tt = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
+                if (col0 + c < dv) tm_cp_async<16>(bv + tt * COLS + c, v + ((size_t)(t0 + tt) * H + h) * dv + col0 + c);
             }
         } else {
-            for (int i = threadIdx.x; i < n * DKP; i += TS_THREADS) {
+            for (int i = threadIdx.x; i < n * DKP; i += THREADS) {
                 const int tt = i / DKP, c = i % DKP;
                 if (c < dk) {
                     const size_t at = ((size_t)(t0 + tt) * H + h) * dk + c;
@@ -338,19 +360,24 @@ time_scan_kernel(const float* __restrict__ r, const float* __restrict__ k, const
                     tm_cp_async<4>(bf + i, fade + at);
                 }
             }
-            for (int i = threadIdx.x; i < n * COLS; i += TS_THREADS) {
+            for (int i = threadIdx.x; i < n * COLS; i += THREADS) {
                 const int tt = i / COLS, c = i % COLS;
                 if (col0 + c < dv) tm_cp_async<4>(bv + i, v + ((size_t)(t0 + tt) * H + h) * dv + col0 + c);
             }
         }
-        if (threadIdx.x < n) tm_cp_async<4>(bb + threadIdx.x, bonus + (size_t)(t0 + threadIdx.x) * H + h);
+        for (int i = threadIdx.x; i < n; i += THREADS) tm_cp_async<4>(bb + i, bonus + (size_t)(t0 + i) * H + h);
     };
     dd_grid_wait();
-    float* sp = state + (((size_t)entry_slot[e] * H + h) * dv + (live ? col : 0)) * DKP + sub * 8;
-    float s[8];
-    {
-        const float4 a = *reinterpret_cast<const float4*>(sp), b = *reinterpret_cast<const float4*>(sp + 4);
-        s[0] = a.x; s[1] = a.y; s[2] = a.z; s[3] = a.w; s[4] = b.x; s[5] = b.y; s[6] = b.z; s[7] = b.w;
+    float* sp = state + ((size_t)entry_slot[e] * H + h) * dv * DKP + sub * 4;
+    float s[C][R];
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+        const int col = min(col0 + my_col + c, dv - 1);
+#pragma unroll
+        for (int p = 0; p < P; ++p) {
+            const float4 x = *reinterpret_cast<const float4*>(sp + (size_t)col * DKP + p * 4 * LPC);
+            s[c][4 * p] = x.x; s[c][4 * p + 1] = x.y; s[c][4 * p + 2] = x.z; s[c][4 * p + 3] = x.w;
+        }
     }
     __syncthreads();                                    // the zeros are written before any copy lands
     if (start < end) stage(start, 0);
@@ -362,7 +389,7 @@ time_scan_kernel(const float* __restrict__ r, const float* __restrict__ k, const
             if (t0 + 2 * TS_TOKENS > end) {             // the last, shorter run: its buffer holds older tokens behind it
                 float* b = staged + (buf ^ 1) * BUF;
                 const int left = end - t0 - TS_TOKENS;
-                for (int i = threadIdx.x + left * DKP; i < TS_TOKENS * DKP; i += TS_THREADS) {
+                for (int i = threadIdx.x + left * DKP; i < TS_TOKENS * DKP; i += THREADS) {
                     b[i] = 0.f;
                     b[TS_TOKENS * DKP + i] = 0.f;
                     b[2 * TS_TOKENS * DKP + i] = 0.f;
@@ -373,36 +400,71 @@ time_scan_kernel(const float* __restrict__ r, const float* __restrict__ k, const
         asm volatile("cp.async.commit_group;" ::: "memory");
         asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
-        const float* sr = staged + buf * BUF + sub * 8;
-        const float* sk = sr + TS_TOKENS * DKP;
-        const float* sf = sk + TS_TOKENS * DKP;
+        const float* sr = staged + buf * BUF + sub * 4;
         const float* sv = staged + buf * BUF + 3 * TS_TOKENS * DKP + my_col;
         const float* sb = staged + buf * BUF + TS_TOKENS * (3 * DKP + COLS);
-#pragma unroll 1
-        for (int tt0 = 0; tt0 < n; tt0 += 4) {
-            float read[4], vv[4];
+        // A token's operands are requested while the token before is worked through.
+        float ops[2][3][R], vv[2][C];
+        auto fetch = [&](int tt, int slot) {
+#pragma unroll
+            for (int w = 0; w < 3; ++w)
+#pragma unroll
+                for (int p = 0; p < P; ++p) {
+                    const float4 x = *reinterpret_cast<const float4*>(sr + (w * TS_TOKENS + tt) * DKP + p * 4 * LPC);
+                    ops[slot][w][4 * p] = x.x; ops[slot][w][4 * p + 1] = x.y; ops[slot][w][4 * p + 2] = x.z; ops[slot][w][4 * p + 3] = x.w;
+                }
+#pragma unroll
+            for (int c = 0; c < C; ++c) vv[slot][c] = sv[tt * COLS + c];
+        };
+        fetch(0, 0);
+        // (all sixteen, tokens of zeros among them: one group's exchanges then lie under the next group's products)
+#pragma unroll
+        for (int tt0 = 0; tt0 < TS_TOKENS; tt0 += 4) {
+            float read[4 * C];                          // index token * C + column
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                const int tt = tt0 + j;
-                vv[j] = sv[tt * COLS];
-                read[j] = time_token(s, sr + tt * DKP, sk + tt * DKP, sf + tt * DKP, vv[j]);
+                const int slot = j & 1;
+                fetch(min(tt0 + j + 1, TS_TOKENS - 1), slot ^ 1);
+#pragma unroll
+                for (int c = 0; c < C; ++c) {
+                    float part[P];
+#pragma unroll
+                    for (int p = 0; p < P; ++p) {
+                        part[p] = 0.f;
+#pragma unroll
+                        for (int i = 4 * p; i < 4 * p + 4; ++i) part[p] = __fmaf_rn(s[c][i], ops[slot][0][i], part[p]);
+                    }
+                    read[j * C + c] = part[0];
+#pragma unroll
+                    for (int p = 1; p < P; ++p) read[j * C + c] = __fadd_rn(read[j * C + c], part[p]);
+#pragma unroll
+                    for (int i = 0; i < R; ++i)
+                        s[c][i] = __fmaf_rn(ops[slot][1][i], vv[slot][c], __fmaf_rn(-ops[slot][2][i], s[c][i], s[c][i]));
+                }
             }
+            const int first = spread_sums<4 * C, 1, LPC>(read, sub);
+            constexpr int MINE = 4 * C / LPC > 1 ? 4 * C / LPC : 1;      // sums a lane is left with
+            const bool writes = LPC <= 4 * C || sub < 4 * C;            // (more lanes than sums: the others hold copies)
 #pragma unroll
-            for (int o = LPC / 2; o > 0; o >>= 1) {
-#pragma unroll
-                for (int j = 0; j < 4; ++j) read[j] += __shfl_xor_sync(0xffffffffu, read[j], o);
+            for (int i = 0; i < MINE; ++i) {
+                const int tt = tt0 + (first + i) / C, c = (first + i) % C;
+                const int col = col0 + my_col + c;
+                if (writes && tt < n && col < dv)
+                    out[((size_t)(t0 + tt) * H + h) * dv + col] = __fmaf_rn(sb[tt], sv[tt * COLS + c], read[i]);
             }
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-                if (tt0 + j < n && live && sub == 0)
-                    out[((size_t)(t0 + tt0 + j) * H + h) * dv + col] = __fmaf_rn(sb[tt0 + j], vv[j], read[j]);
         }
         __syncthreads();                                // all have read this buffer before the copies after next fill it
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    if (live && start < end) {
-        *reinterpret_cast<float4*>(sp) = make_float4(s[0], s[1], s[2], s[3]);
-        *reinterpret_cast<float4*>(sp + 4) = make_float4(s[4], s[5], s[6], s[7]);
+    if (start < end) {
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+            const int col = col0 + my_col + c;
+            if (col >= dv) continue;
+#pragma unroll
+            for (int p = 0; p < P; ++p)
+                *reinterpret_cast<float4*>(sp + (size_t)col * DKP + p * 4 * LPC) = make_float4(s[c][4 * p], s[c][4 * p + 1], s[c][4 * p + 2], s[c][4 * p + 3]);
+        }
     }
 }
 
@@ -539,23 +601,23 @@ DD_API int dd_time_scan(const float* r, const float* k, const float* v, const fl
     if (((uintptr_t)r | (uintptr_t)k | (uintptr_t)v | (uintptr_t)fade | (uintptr_t)state) & 15)
         return dd_fail("dd_time_scan: operands must be 16-byte aligned");
     cudaStream_t s = (cudaStream_t)stream;
-    const int lpc = lanes_of(dk), cols = TS_THREADS / lpc;
-    const dim3 grid(dd_ceil_div(dv, cols), H, n_entries);
-    const size_t smem = (size_t)2 * (TS_TOKENS * (3 * 8 * lpc + cols + 1)) * sizeof(float);
-#define DD_SCAN(L)                                                                                                      \
+    // blocks of 16 columns (more where a warp holds more)
+#define DD_SCAN(R, C, L)                                                                                                \
     do {                                                                                                                \
+        constexpr int TH = L * 16 / C > 32 ? L * 16 / C : 32, COLS = TH / L * C;                                        \
+        const size_t smem = (size_t)2 * (TS_TOKENS * (3 * R * L + COLS + 1)) * sizeof(float);                           \
         if (smem > 48 * 1024)                                                                                           \
-            cudaFuncSetAttribute(time_scan_kernel<L>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
-        dd_launch_in_order(time_scan_kernel<L>, grid, dim3(TS_THREADS), smem, s, r, k, v, fade, bonus, entry_start, entry_slot, \
-                           state, out, H, dk, dv);                                                                      \
+            cudaFuncSetAttribute(time_scan_kernel<R, C, L, TH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        dd_launch_in_order(time_scan_kernel<R, C, L, TH>, dim3(dd_ceil_div(dv, COLS), H, n_entries), dim3(TH), smem, s, r, k, v, \
+                           fade, bonus, entry_start, entry_slot, state, out, H, dk, dv);                                \
     } while (0)
-    switch (lpc) {
-        case 1: DD_SCAN(1); break;
-        case 2: DD_SCAN(2); break;
-        case 4: DD_SCAN(4); break;
-        case 8: DD_SCAN(8); break;
-        case 16: DD_SCAN(16); break;
-        default: DD_SCAN(32); break;
+    switch (8 * lanes_of(dk)) {
+        case 8: DD_SCAN(4, 4, 2); break;
+        case 16: DD_SCAN(4, 4, 4); break;
+        case 32: DD_SCAN(4, 4, 8); break;
+        case 64: DD_SCAN(4, 4, 16); break;
+        case 128: DD_SCAN(4, 4, 32); break;
+        default: DD_SCAN(8, 2, 32); break;
     }
 #undef DD_SCAN
     return dd_check_launch("dd_time_scan");
