@@ -14,7 +14,7 @@ __global__ void __launch_bounds__(THREADS)
 gemm_simt_kernel(const TI* __restrict__ A, int lda, const TI* __restrict__ W, int ldw,
                  const float* __restrict__ bias, const float* residual, int ldr,
                  TO* C, int ldc, int M, int N, int K, int act,
-                 const int* __restrict__ tile_group, long long group_stride) {
+                 const int* __restrict__ tile_group, long long group_stride, const float* __restrict__ row_scale) {
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[BK][BN + 4];
     dd_launch_dependents();
@@ -67,6 +67,7 @@ gemm_simt_kernel(const TI* __restrict__ A, int lda, const TI* __restrict__ W, in
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
+            if (row_scale) v *= row_scale[m];
             if (bias) v += bias[n];
             v = dd_activation(v, act);
             if (residual) v += residual[(size_t)m * ldr + n];
@@ -275,17 +276,17 @@ int launch(const void* A, int lda, const void* W, int ldw, const float* bias, co
     dim3 grid(dd_ceil_div(N, BN), dd_ceil_div(M, BM));
     if (grid.y > 65535) return dd_fail("dd_gemm_simt: too many rows (%d)", M);
     dd_launch(gemm_simt_kernel<TI, TO>, dim3(grid), dim3(THREADS), 0, s, (const TI*)A, lda, (const TI*)W, ldw, bias, residual, ldr,
-                                                     (TO*)C, ldc, M, N, K, act, (const int*)nullptr, 0LL);
+                                                     (TO*)C, ldc, M, N, K, act, (const int*)nullptr, 0LL, (const float*)nullptr);
     return dd_check_launch("dd_gemm_simt");
 }
 
 template <typename TI, typename TO>
 int launch_grouped(const void* A, int lda, const void* W, int ldw, long long group_stride, const int* tile_group,
-                   void* C, int ldc, int M, int N, int K, int act, cudaStream_t s) {
+                   void* C, int ldc, int M, int N, int K, int act, cudaStream_t s, const float* row_scale) {
     dim3 grid(dd_ceil_div(N, BN), dd_ceil_div(M, BM));
     if (grid.y > 65535) return dd_fail("dd_gemm_simt_grouped: too many rows (%d)", M);
     dd_launch(gemm_simt_kernel<TI, TO>, dim3(grid), dim3(THREADS), 0, s, (const TI*)A, lda, (const TI*)W, ldw,
-              (const float*)nullptr, (const float*)nullptr, 0, (TO*)C, ldc, M, N, K, act, tile_group, group_stride);
+              (const float*)nullptr, (const float*)nullptr, 0, (TO*)C, ldc, M, N, K, act, tile_group, group_stride, row_scale);
     return dd_check_launch("dd_gemm_simt_grouped");
 }
 }  // namespace
@@ -295,20 +296,21 @@ DD_API int dd_gemm_simt_group_tile() { return BM; }
 
 // Grouped product: W is a stack of matrices [groups][N, K] (group_stride elements apart, rows ldw apart); the rows
 // of A come in tiles of dd_gemm_simt_group_tile() rows, tile i multiplied with matrix tile_group[i] (a device array
-// of ceil(M / tile) entries; -1: the tile holds no rows and is skipped, its rows of C are left as they are).
+// of ceil(M / tile) entries; -1: the tile holds no rows and is skipped, its rows of C are left as they are). row_scale: float32 [M]
+// or null; a row's sums are multiplied by it before the activation.
 // The arithmetic per output element is that of dd_gemm_simt (k ascending, fmaf from zero).
 DD_API int dd_gemm_simt_grouped(const void* A, int lda, const void* W, int ldw, long long group_stride,
                                 const int* tile_group, void* C, int ldc, int M, int N, int K, int act,
-                                int in_dtype, int out_dtype, void* stream) {
+                                int in_dtype, int out_dtype, void* stream, const float* row_scale) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || !tile_group) return dd_fail("dd_gemm_simt_grouped: bad K=%d or no tile groups", K);
     cudaStream_t s = (cudaStream_t)stream;
     if (in_dtype == DD_F32 && out_dtype == DD_F32)
-        return launch_grouped<float, float>(A, lda, W, ldw, group_stride, tile_group, C, ldc, M, N, K, act, s);
+        return launch_grouped<float, float>(A, lda, W, ldw, group_stride, tile_group, C, ldc, M, N, K, act, s, row_scale);
     if (in_dtype == DD_BF16 && out_dtype == DD_F32)
-        return launch_grouped<__nv_bfloat16, float>(A, lda, W, ldw, group_stride, tile_group, C, ldc, M, N, K, act, s);
+        return launch_grouped<__nv_bfloat16, float>(A, lda, W, ldw, group_stride, tile_group, C, ldc, M, N, K, act, s, row_scale);
     if (in_dtype == DD_BF16 && out_dtype == DD_BF16)
-        return launch_grouped<__nv_bfloat16, __nv_bfloat16>(A, lda, W, ldw, group_stride, tile_group, C, ldc, M, N, K, act, s);
+        return launch_grouped<__nv_bfloat16, __nv_bfloat16>(A, lda, W, ldw, group_stride, tile_group, C, ldc, M, N, K, act, s, row_scale);
     return dd_fail("dd_gemm_simt_grouped: unsupported dtypes in=%d out=%d", in_dtype, out_dtype);
 }
 

@@ -6,7 +6,8 @@
 //
 //   dd_route_by_table   token ids + table [vocab, K] -> pair_row [N*K] (the row of pair (t, k); -2 for an
 //                       identity expert, whose output is the token's own input row: experts n_experts .. n_experts +
-//                       n_identity - 1 of the table; they have no rows), row_token [rows]
+//                       n_identity - 1 of the table; they have no rows), row_token [rows]; with pair_weight
+//                       [N*K] also row_weight [rows], a row's weight (0 for a row of padding)
 //                       (the token of a row, -1 for a row of padding), tile_group [rows / tile]
 //   dd_gather_rows      x [N, width] -> sorted rows (a row of padding is zeroed)
 //                       (ids null: token t reads row t of the table, which then holds the step's own choices)
@@ -29,7 +30,8 @@ constexpr int ROUTE_THREADS = 1024;
 __global__ void __launch_bounds__(ROUTE_THREADS)
 route_by_table_kernel(const int* __restrict__ ids, const int* __restrict__ table, int n_tokens, int vocab, int top,
                       int n_experts, int tile, int n_rows, int* __restrict__ pair_row, int* __restrict__ row_token,
-                      int* __restrict__ tile_group, int* __restrict__ error_flag, int n_identity) {
+                      int* __restrict__ tile_group, int* __restrict__ error_flag, int n_identity,
+                      const float* __restrict__ pair_weight, float* __restrict__ row_weight) {
     extern __shared__ int shared[];              // [E] counts, then cursors; [E + 1] first rows
     int* count = shared;
     int* first = shared + n_experts;
@@ -37,7 +39,10 @@ route_by_table_kernel(const int* __restrict__ ids, const int* __restrict__ table
     dd_grid_wait();
     const int n_pairs = n_tokens * top;
     for (int e = threadIdx.x; e < n_experts; e += ROUTE_THREADS) count[e] = 0;
-    for (int r = threadIdx.x; r < n_rows; r += ROUTE_THREADS) row_token[r] = -1;
+    for (int r = threadIdx.x; r < n_rows; r += ROUTE_THREADS) {
+        row_token[r] = -1;
+        if (row_weight) row_weight[r] = 0.f;
+    }
     for (int i = threadIdx.x; i < n_rows / tile; i += ROUTE_THREADS) tile_group[i] = -1;
     __syncthreads();
     // four pairs of a thread at a time: their token ids are requested together, then their table entries (one pair
@@ -93,6 +98,7 @@ route_by_table_kernel(const int* __restrict__ ids, const int* __restrict__ table
             const int row = first[e[u]] + atomicAdd(&count[e[u]], 1);
             pair_row[pair] = row;
             row_token[row] = pair / top;
+            if (row_weight) row_weight[row] = pair_weight[pair];
         }
     }
 }
@@ -371,7 +377,7 @@ combine_rows_kernel(const float* __restrict__ y, const int* __restrict__ pair_ro
 // * (tile - 1): every expert that has a pair may waste all but one row of its last tile. A token id or a table entry out of range sets error bit 1 and leaves its pair out.
 DD_API int dd_route_by_table(const int* ids, const int* table, int n_tokens, int vocab, int top, int n_experts, int tile,
                              int n_rows, int* pair_row, int* row_token, int* tile_group, int* error_flag, void* stream,
-                             int n_identity) {
+                             int n_identity, const float* pair_weight, float* row_weight) {
     if (n_tokens <= 0) return 0;
     const long long n_pairs = (long long)n_tokens * top;
     if (top <= 0 || n_experts <= 0 || tile <= 0 || n_rows % tile ||
@@ -380,7 +386,7 @@ DD_API int dd_route_by_table(const int* ids, const int* table, int n_tokens, int
                        n_tokens, top, n_experts);
     if (n_experts > 8192) return dd_fail("dd_route_by_table: %d experts are more than a block counts", n_experts);
     dd_launch(route_by_table_kernel, dim3(1), dim3(ROUTE_THREADS), (size_t)(2 * n_experts + 1) * sizeof(int), (cudaStream_t)stream,
-              ids, table, n_tokens, vocab, top, n_experts, tile, n_rows, pair_row, row_token, tile_group, error_flag, n_identity);
+              ids, table, n_tokens, vocab, top, n_experts, tile, n_rows, pair_row, row_token, tile_group, error_flag, n_identity, pair_weight, row_weight);
     return dd_check_launch("dd_route_by_table");
 }
 

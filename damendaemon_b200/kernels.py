@@ -50,8 +50,8 @@ _SIGNATURES = {
         "dd_time_step": [_c_void] * 4 + [_c_int] + [_c_void] * 4 + [_c_float, _c_void, _c_int, _c_void, _c_void] + [_c_int] * 5 + [_c_void],
         "dd_rotary": [_c_void, _c_void, _c_int, _c_void, _c_void, _c_float] + [_c_int] * 7 + [_c_void],
         "dd_gemm_simt_group_tile": [],
-        "dd_gemm_simt_grouped": [_c_void, _c_int, _c_void, _c_int, ctypes.c_longlong, _c_void, _c_void, _c_int] + [_c_int] * 6 + [_c_void],
-        "dd_route_by_table": [_c_void, _c_void] + [_c_int] * 6 + [_c_void] * 5 + [_c_int],
+        "dd_gemm_simt_grouped": [_c_void, _c_int, _c_void, _c_int, ctypes.c_longlong, _c_void, _c_void, _c_int] + [_c_int] * 6 + [_c_void, _c_void],
+        "dd_route_by_table": [_c_void, _c_void] + [_c_int] * 6 + [_c_void] * 5 + [_c_int, _c_void, _c_void],
         "dd_gather_rows": [_c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void],
         "dd_gated_unit": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void, _c_int, _c_void],
         "dd_combine_rows": [_c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_float, _c_void, _c_void, _c_void, _c_int],
@@ -86,13 +86,22 @@ _SIGNATURES = {
         "dd_recurrence_gates": [_c_void] * 6 + [_c_float, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void],
         "dd_linear_scan": [_c_void, _c_void, _c_void, _c_int, _c_void, _c_void, _c_int, _c_void, _c_void, _c_int, _c_int, _c_int,
                            _c_int, _c_void],
+        "dd_memory_gates": [_c_void, _c_int, _c_float, _c_void, _c_void, _c_int] + [_c_void] * 4 + [_c_int, _c_void],
+        "dd_memory_prepare": [_c_void, _c_void, _c_void, _c_int, _c_float, _c_int] + [_c_void] * 4 + [_c_int] * 6 + [_c_void],
+        "dd_memory_scan": [_c_void] * 7 + [_c_int, _c_void, _c_void] + [_c_int] * 4 + [_c_void],
+        "dd_memory_step": [_c_void] * 4 + [_c_int, _c_float, _c_int, _c_void, _c_int, _c_float, _c_void, _c_void, _c_void, _c_int, _c_void,
+                           _c_void, _c_float, _c_float, _c_void, _c_int, _c_void, _c_void] + [_c_int] * 5 + [_c_void],
+        "dd_memory_finish": [_c_void, _c_void, _c_void, _c_int, _c_void, _c_float, _c_float, _c_int, _c_void, _c_int] + [_c_int] * 4 + [_c_void],
+        "dd_post_norm": [_c_void, _c_void, _c_void, _c_float, _c_float, _c_void, _c_int, _c_void, _c_float, _c_float, _c_void, _c_int,
+                         _c_int, _c_int, _c_void],
+        "dd_round_rows": [_c_void, _c_void, ctypes.c_longlong, _c_void],
         "dd_sample": [_c_void, _c_int, _c_int, _c_int] + [_c_void] * 6,
         "dd_adjust_logits": [_c_void, _c_int, _c_int] + [_c_void] * 8 + [_c_int, _c_void],
     },
     "tensor": {
         "dd_gemm_tcgen05_plan": [_c_int, _c_int, _c_int, _c_int, _c_void, _c_void],
         "dd_gemm_grouped_tcgen05": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int] + [_c_int] * 5
-                                   + [_c_float, _c_float, _c_int, _c_void, _c_void, _c_int],
+                                   + [_c_float, _c_float, _c_int, _c_void, _c_void, _c_int, _c_int, _c_void],
         "dd_wait_probe": [ctypes.c_ulonglong, _c_void, _c_void, _c_void],
         "dd_attention_decode_supported": [_c_int] * 4,
         "dd_attention_prefill_supported": [_c_int] * 4,
@@ -497,6 +506,172 @@ def linear_scan(a, drive, y, entry_start, entry_slot, state, activation=None, ou
     _call(library("core"), "dd_linear_scan", _ptr(a), _ptr(drive), _ptr(y, "y"), y.stride(0),
           _ptr(entry_start, "entry_start", torch.int32), _ptr(entry_slot, "entry_slot", torch.int32), entry_slot.numel(), _ptr(state),
           _ptr(out), out.stride(0), width, {None: 0, "gelu_tanh": 1}[activation], _dt(y.dtype), _stream())
+    return out
+
+
+def memory_state_shape(heads, head_dim, value_dim, gated):
+    """Shape of one request's matrix memory (float32): per head the columns of S one after the other (and, gated, the vector n
+    as one more column), each padded to eight rows times a power of two; zeros for a new request."""
+    if not 0 < head_dim <= 256 or not 0 < value_dim <= 4096:
+        raise KernelError(f"matrix memory: heads of {head_dim} by {value_dim} are not supported (keys of at most 256, values of at most 4096)")
+    lanes = 1
+    while lanes * 8 < head_dim:
+        lanes *= 2
+    return (int(heads), int(value_dim) + (1 if gated else 0), 8 * lanes)
+
+
+def _up4(n):
+    return -(-n // 4) * 4
+
+
+def memory_gates(z, cap, entry_start, entry_slot, peak):
+    """The gates of a step from their projections z (float32 row view [N, 2 * heads]: input gates, then forget gates): with
+    i = cap tanh(z_i / cap), f = log sigmoid(cap tanh(z_f / cap)) and, token by token from row entry_slot[e] of ``peak``
+    (float32 [slots, heads], read and written), M' = max(f + M, i): (fade = 1 - exp(f + M - M'), take = exp(i - M'), floor =
+    exp(-M')), float32 [N, heads] each."""
+    n, heads = z.shape[0], z.shape[1] // 2
+    if z.dtype != torch.float32 or z.stride(1) != 1 or z.shape[1] != 2 * heads or peak.dtype != torch.float32 or \
+            not peak.is_contiguous() or tuple(peak.shape[1:]) != (heads,):
+        raise KernelError("memory_gates: shapes do not fit")
+    fade, take, floor = (torch.empty((n, heads), dtype=torch.float32, device=z.device) for _ in range(3))
+    _call(library("core"), "dd_memory_gates", _ptr(z, "z"), z.stride(0), float(cap), _ptr(entry_start, "entry_start", torch.int32),
+          _ptr(entry_slot, "entry_slot", torch.int32), entry_slot.numel(), _ptr(peak), _ptr(fade), _ptr(take), _ptr(floor), heads, _stream())
+    return fade, take, floor
+
+
+def _memory_operands(q, k, v, heads, head_dim, value_dim, *more):
+    n = q.shape[0]
+    if q.shape != (n, heads * head_dim) or k.shape != q.shape or v.shape != (n, heads * value_dim) or \
+            any(t.stride(0) != q.stride(0) or t.stride(1) != 1 or t.dtype != q.dtype for t in (q, k, v, *more)) or \
+            any(t.shape != v.shape for t in more):
+        raise KernelError("matrix memory: the operands do not fit the heads (row views of one stride and type)")
+    return n
+
+
+def memory_prepare(q, k, v, heads, head_dim, value_dim, scale=1.0, silu=False, take=None):
+    """The recurrence's operands as float32 rows, each head's padded to a multiple of four: (q * scale [N, heads, .], k * take
+    [N, heads, .], v [N, heads, .]), q, k and v through silu first if asked. take (float32 [N, heads] or None) also appends the
+    column of ones to v. q, k, v: row views of one buffer."""
+    n = _memory_operands(q, k, v, heads, head_dim, value_dim)
+    if take is not None and (take.shape != (n, heads) or take.dtype != torch.float32 or not take.is_contiguous()):
+        raise KernelError("memory_prepare: take must be float32 [N, heads]")
+    ones = 0 if take is None else 1
+    f32 = lambda w: torch.empty((n, heads, _up4(w)), dtype=torch.float32, device=q.device)
+    qo, ko, vo = f32(head_dim), f32(head_dim), f32(value_dim + ones)
+    _call(library("core"), "dd_memory_prepare", _ptr(q, "q"), _ptr(k, "k"), _ptr(v, "v"), q.stride(0), float(scale), 1 if silu else 0,
+          _ptr(take, "take"), _ptr(qo), _ptr(ko), _ptr(vo), n, heads, head_dim, value_dim, ones, _dt(q.dtype), _stream())
+    return qo, ko, vo
+
+
+def memory_scan(q, k, v, fade, entry_start, entry_slot, state, head_dim, value_dim, out=None):
+    """The recurrence of a step: per entry and head, from row entry_slot[e] of ``state`` (float32 [slots,
+    *memory_state_shape(...)], read and written), token by token: S = S - fade * S + k v^T; o = S^T q. fade: float32 [N, heads]
+    (gated: the state has a column n and v its ones), or [heads] (the same for every token). Returns o float32 [N, heads,
+    value_dim (+ 1) rounded up to four]."""
+    n, heads = q.shape[0], q.shape[1]
+    per_token = fade.dim() == 2
+    ones = 1 if per_token else 0
+    ok = all(t.dtype == torch.float32 and t.is_contiguous() for t in (q, k, v, fade, state))
+    if not ok or q.shape[2] != _up4(head_dim) or k.shape != q.shape or v.shape != (n, heads, _up4(value_dim + ones)) or \
+            fade.shape != ((n, heads) if per_token else (heads,)) or \
+            tuple(state.shape[1:]) != memory_state_shape(heads, head_dim, value_dim, per_token):
+        raise KernelError("memory_scan: shapes do not fit the state")
+    if out is None:
+        out = torch.empty(v.shape, dtype=torch.float32, device=q.device)
+    _call(library("core"), "dd_memory_scan", _ptr(q), _ptr(k), _ptr(v), _ptr(fade) if per_token else None,
+          None if per_token else _ptr(fade), _ptr(entry_start, "entry_start", torch.int32), _ptr(entry_slot, "entry_slot", torch.int32),
+          entry_slot.numel(), _ptr(state), _ptr(out), heads, head_dim, value_dim, ones, _stream())
+    return out
+
+
+def memory_slices(entries, heads, head_dim, value_dim, device):
+    """Into how many blocks ``memory_step`` cuts a head's columns: as many as fill the GPU about twice, while a block keeps at
+    least the columns its threads hold at once."""
+    lanes = memory_state_shape(heads, head_dim, value_dim, False)[2] // 8
+    slices = 1
+    while slices < 8 and entries * heads * slices * 2 <= 2 * sm_count(device) and value_dim >= 2 * slices * max(1, 256 // lanes):
+        slices *= 2
+    return slices
+
+
+def memory_step(q, k, v, gate, entry_slot, state, heads, head_dim, value_dim, weight=None, eps=0.0, den_eps=0.0, scale=1.0, silu=False,
+                gates=None, fade=None, slices=None, out=None):
+    """A step of single tokens (row e is entry e) in one kernel. gates = (z, cap, peak) as ``memory_gates`` takes them, or fade
+    float32 [heads]. weight (float32 [heads * value_dim]) given: ``memory_finish`` with a norm per head is part of it and [N,
+    heads * value_dim] in q's type is returned; None: (o, floor) as ``memory_scan`` and ``memory_gates`` leave them (floor None
+    without gates)."""
+    n = _memory_operands(q, k, v, heads, head_dim, value_dim, *(() if gate is None else (gate,)))
+    gated = gates is not None
+    if state.dtype != torch.float32 or not state.is_contiguous() or entry_slot.numel() != n or gated == (fade is not None) or \
+            tuple(state.shape[1:]) != memory_state_shape(heads, head_dim, value_dim, gated) or (weight is not None and (
+                gate is None or weight.numel() != heads * value_dim or weight.dtype != torch.float32 or not weight.is_contiguous())):
+        raise KernelError("memory_step: shapes do not fit the state")
+    z = peak = None
+    cap = 0.0
+    if gated:
+        z, cap, peak = gates
+        if z.dtype != torch.float32 or z.shape != (n, 2 * heads) or z.stride(1) != 1 or peak.dtype != torch.float32 or \
+                not peak.is_contiguous() or tuple(peak.shape[1:]) != (heads,):
+            raise KernelError("memory_step: the gates do not fit")
+    elif fade.shape != (heads,) or fade.dtype != torch.float32:
+        raise KernelError("memory_step: fade must be float32 [heads]")
+    o = floor = None
+    if weight is not None:
+        if out is None:
+            out = torch.empty((n, heads * value_dim), dtype=q.dtype, device=q.device)
+    else:
+        o = torch.empty((n, heads, _up4(value_dim + (1 if gated else 0))), dtype=torch.float32, device=q.device)
+        floor = torch.empty((n, heads), dtype=torch.float32, device=q.device) if gated else None
+    _call(library("core"), "dd_memory_step", _ptr(q, "q"), _ptr(k, "k"), _ptr(v, "v"), _ptr(gate, "gate"), q.stride(0), float(scale),
+          1 if silu else 0, _ptr(z, "z"), 0 if z is None else z.stride(0), float(cap), _ptr(fade, "fade"), _ptr(peak, "peak"),
+          _ptr(entry_slot, "entry_slot", torch.int32), n, _ptr(state), _ptr(weight, "weight"), float(eps), float(den_eps), _ptr(out),
+          0 if out is None else out.stride(0), _ptr(o), _ptr(floor), heads, head_dim, value_dim,
+          memory_slices(n, heads, head_dim, value_dim, q.device) if slices is None else int(slices), _dt(q.dtype), _stream())
+    return out if weight is not None else (o, floor)
+
+
+def memory_finish(o, gate, weight, heads, value_dim, eps, den_eps=0.0, floor=None, together=False, out=None):
+    """x = o, over max(|n . q|, floor) + den_eps where floor (float32 [N, heads]) is given (n . q is element value_dim of a head's
+    row); out = x / sqrt(mean(x^2) + eps) * weight * sigmoid(gate), the mean over every head, or over all heads together. o as
+    ``memory_scan`` leaves it; gate a row view [N, heads * value_dim], whose type out has; weight float32 [heads * value_dim]."""
+    n = o.shape[0]
+    if o.dtype != torch.float32 or not o.is_contiguous() or o.shape != (n, heads, _up4(value_dim + (0 if floor is None else 1))) or \
+            gate.shape != (n, heads * value_dim) or gate.stride(1) != 1 or weight.numel() != heads * value_dim or \
+            weight.dtype != torch.float32 or not weight.is_contiguous() or (floor is not None and (
+                floor.shape != (n, heads) or floor.dtype != torch.float32 or not floor.is_contiguous())):
+        raise KernelError("memory_finish: the gate, the weight or the floor does not fit the read-out")
+    if out is None:
+        out = torch.empty((n, heads * value_dim), dtype=gate.dtype, device=o.device)
+    _call(library("core"), "dd_memory_finish", _ptr(o), _ptr(floor, "floor"), _ptr(gate, "gate"), gate.stride(0), _ptr(weight, "weight"),
+          float(eps), float(den_eps), 1 if together else 0, _ptr(out), out.stride(0), n, heads, value_dim, _dt(gate.dtype), _stream())
+    return out
+
+
+def post_norm(x, a, weight=None, eps=0.0, factor=1.0, scale=1.0, other=None, other_scale=1.0, pair_row=None, rounded_dtype=None):
+    """In place x += factor * y / sqrt(mean(y^2) + eps) * weight (weight None: x += factor * y), with y = scale * a + other_scale *
+    other, or, with pair_row (int32 [N * top], as ``route_by_table`` leaves it), y[t] = the sum of a's rows at the token's
+    entries. x, a, other: float32 contiguous rows of one width. Returns x rounded to rounded_dtype (None without one)."""
+    n, width = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or a.dtype != torch.float32 or not a.is_contiguous() or a.shape[1] != width or \
+            (pair_row is None and a.shape[0] != n) or (pair_row is not None and (pair_row.numel() % max(1, n) or other is not None)) or \
+            (other is not None and (other.shape != x.shape or other.dtype != torch.float32 or not other.is_contiguous())) or \
+            (weight is not None and (weight.numel() != width or weight.dtype != torch.float32 or not weight.is_contiguous())):
+        raise KernelError("post_norm: float32 rows of one width and a float32 weight of it wanted")
+    rounded = None if rounded_dtype is None else torch.empty((n, width), dtype=rounded_dtype, device=x.device)
+    _call(library("core"), "dd_post_norm", _ptr(x, "x"), _ptr(a, "a"), _ptr(other, "other"), float(scale), float(other_scale),
+          _ptr(pair_row, "pair_row", torch.int32), 0 if pair_row is None else pair_row.numel() // n, _ptr(weight, "weight"), float(eps),
+          float(factor), _ptr(rounded), n, width, _dt(rounded_dtype or torch.float32), _stream())
+    return rounded
+
+
+def round_rows(x, dtype):
+    """x (float32, contiguous) in ``dtype``: x itself where that is float32."""
+    if dtype == torch.float32:
+        return x
+    if x.dtype != torch.float32 or not x.is_contiguous() or dtype != torch.bfloat16:
+        raise KernelError("round_rows: contiguous float32 rows to bfloat16 wanted")
+    out = torch.empty(x.shape, dtype=dtype, device=x.device)
+    _call(library("core"), "dd_round_rows", _ptr(x, "x"), _ptr(out), x.numel(), _stream())
     return out
 
 
@@ -1039,21 +1214,27 @@ def grouped_rows(n_tokens, top, n_experts, tile):
     return -(-(pairs + min(n_experts, pairs) * (tile - 1)) // tile) * tile
 
 
-def route_by_table(ids, table, n_experts, tile, n_identity=0):
+def route_by_table(ids, table, n_experts, tile, n_identity=0, pair_weight=None):
     """ids int32 [N], table int32 [vocab, K] -> (pair_row [N*K], row_token [rows], tile_group [rows/tile]). ids None:
     token t reads row t of the table (the step's own choices, [N, K], as ``route_by_score`` leaves them). Table entries
     n_experts .. n_experts + n_identity - 1 are experts whose output is the token's own input: they get no rows, their pairs
-    the pair_row -2 (see ``combine_rows``)."""
+    the pair_row -2 (see ``combine_rows``). pair_weight: float32 [N * K] or None; given, a fourth result row_weight [rows] holds
+    every row's weight (0 for a row of padding)."""
     vocab, top = table.shape
     n = vocab if ids is None else ids.numel()
     rows = grouped_rows(n, top, n_experts, tile)
     pair_row = torch.empty((n * top,), dtype=torch.int32, device=table.device)
     row_token = torch.empty((rows,), dtype=torch.int32, device=table.device)
     tile_group = torch.empty((rows // tile,), dtype=torch.int32, device=table.device)
+    row_weight = None
+    if pair_weight is not None:
+        if pair_weight.numel() != n * top or pair_weight.dtype != torch.float32 or not pair_weight.is_contiguous():
+            raise KernelError("route_by_table: pair_weight must be float32 [tokens * top]")
+        row_weight = torch.empty((rows,), dtype=torch.float32, device=table.device)
     _call(library("core"), "dd_route_by_table", _ptr(ids, "ids", torch.int32), _ptr(table, "table", torch.int32), n, vocab, top,
           n_experts, tile, rows, _ptr(pair_row), _ptr(row_token), _ptr(tile_group), _ptr(error_flag(table.device)), _stream(),
-          int(n_identity))
-    return pair_row, row_token, tile_group
+          int(n_identity), _ptr(pair_weight, "pair_weight"), _ptr(row_weight))
+    return (pair_row, row_token, tile_group) if row_weight is None else (pair_row, row_token, tile_group, row_weight)
 
 
 def route_by_score(y, router, n_experts, top, groups=1, keep=1, weight_scale=1.0, shared_gate=False, softmax=False,
@@ -1096,9 +1277,15 @@ def simt_group_tile():
     return int(library("core").dd_gemm_simt_group_tile())
 
 
-def gemm_simt_grouped(a, w, tile_group, activation=None, out_dtype=None):
+def _check_row_scale(row_scale, rows):
+    if row_scale is not None and (row_scale.numel() != rows or row_scale.dtype != torch.float32 or not row_scale.is_contiguous()):
+        raise KernelError("grouped gemm: row_scale must be float32 [rows]")
+
+
+def gemm_simt_grouped(a, w, tile_group, activation=None, out_dtype=None, row_scale=None):
     """a [rows, K] in tiles of simt_group_tile() rows; w [groups, N, K]; tile i is multiplied with w[tile_group[i]]
-    (skipped where that is negative). CUDA-core float32 multiply-add, k ascending."""
+    (skipped where that is negative); act(row_scale[r] * product). CUDA-core float32 multiply-add, k ascending."""
+    _check_row_scale(row_scale, a.shape[0])
     _rows(a, "a")
     if w.dim() != 3 or not w.is_contiguous() or w.shape[2] != a.shape[1] or w.dtype != a.dtype:
         raise KernelError(f"grouped gemm: a {tuple(a.shape)} {a.dtype} does not fit w {tuple(w.shape)} {w.dtype}")
@@ -1108,20 +1295,23 @@ def gemm_simt_grouped(a, w, tile_group, activation=None, out_dtype=None):
     out = torch.empty((M, N), dtype=out_dtype, device=a.device)
     _call(library("core"), "dd_gemm_simt_grouped", _ptr(a, "a"), a.stride(0), _ptr(w, "w"), w.stride(1), w.stride(0),
           _ptr(tile_group, "tile_group", torch.int32), _ptr(out), out.stride(0), M, N, K, ACTIVATIONS[activation],
-          _dt(a.dtype), _dt(out_dtype), _stream())
+          _dt(a.dtype), _dt(out_dtype), _stream(), _ptr(row_scale, "row_scale"))
     return out
 
 
 GROUPED_TCGEN05_TILES = (16, 32, 64, 128)
 
 
-def gemm_grouped_tcgen05(a, w, tile_group, tile, gated=None, out_dtype=None):
+def gemm_grouped_tcgen05(a, w, tile_group, tile, gated=None, out_dtype=None, activation=None, row_scale=None):
     """a [rows, K] bfloat16 in tiles of ``tile`` rows (one of GROUPED_TCGEN05_TILES); w [groups, N, K] bfloat16; tile i
     is multiplied with w[tile_group[i]] on the tensor cores (skipped where that is negative). gated=(limit, alpha) or
     (limit, alpha, form): w holds gate rows then up rows ([groups, 2 * inner, K]) and the result is the gated unit (form:
     one of GATED_FORMS, the clamped one by default) of the two products, [rows, inner], computed in float32 in the
-    product's epilogue."""
+    product's epilogue. Without ``gated``: act(row_scale[r] * product), row_scale float32 [rows] or None, in the epilogue."""
     _rows(a, "a")
+    _check_row_scale(row_scale, a.shape[0])
+    if gated and (activation or row_scale is not None):
+        raise KernelError("grouped gemm: an activation or a row scale does not go with the gated unit")
     if w.dim() != 3 or not w.is_contiguous() or w.shape[2] != a.shape[1] or w.dtype != torch.bfloat16 or a.dtype != torch.bfloat16:
         raise KernelError(f"grouped gemm: a {tuple(a.shape)} {a.dtype} does not fit w {tuple(w.shape)} {w.dtype}")
     rows, K = a.shape
@@ -1132,7 +1322,8 @@ def gemm_grouped_tcgen05(a, w, tile_group, tile, gated=None, out_dtype=None):
     limit, alpha, form = (tuple(gated) + ("clamped_swish",))[:3] if gated else (0.0, 0.0, "clamped_swish")
     _call(library("tensor"), "dd_gemm_grouped_tcgen05", _ptr(a, "a"), a.stride(0), _ptr(w, "w"), w.stride(1), groups, per_group,
           _ptr(tile_group, "tile_group", torch.int32), _ptr(out), out.stride(0), rows, N, K, int(tile), 1 if gated else 0,
-          float(limit), float(alpha), _dt(out_dtype), _ptr(error_flag(a.device)), _stream(), GATED_FORMS[form])
+          float(limit), float(alpha), _dt(out_dtype), _ptr(error_flag(a.device)), _stream(), GATED_FORMS[form],
+          ACTIVATIONS[activation], _ptr(row_scale, "row_scale"))
     return out
 
 

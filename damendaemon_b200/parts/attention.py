@@ -197,5 +197,5 @@ class Attention(Mixer):
         attended = ctx.attend(q, k, v, cache, s.n_heads, s.scale, s.window, gate=None if s.gate_per_element else gate, **self.mask)
         if s.gate_per_element:
             kernels.sigmoid_gate(attended, gate)
-        return linear(self.runtime, attended, self.out_w, self.out_b, residual=residual, out_dtype=residual.dtype,
+        return linear(self.runtime, attended, self.out_w, self.out_b, residual=residual, out_dtype=torch.float32,
                       out=residual)

@@ -9,9 +9,12 @@ that reads blends of its input with the token before gets them from that pass as
 'pre_norm_shift': 'pre_norm' (or, with one norm, 'pre_norm_mixer') whose mixer reads s[t] = n[t] + (n[t-1] - n[t]) * mu
 with n = norm[0](x) and mu one number per channel; n[t-1] of a sequence's first token is zero, and across steps it is kept
 per request (a state named 'shift' at the layer's cache site).
+'post_norm': x = x + c norm[0](mixer(x)); x = x + c norm[1](feed_forward(x)) (with one norm there is no feed-forward): a
+sublayer reads the stream itself, in the engine dtype. Norm, add and the rounding that the next sublayer reads are one pass.
 """
 from __future__ import annotations
 
+from .. import kernels
 from ..cache.manager import RequestState
 from .registry import register_arrangement
 from .spec import TensorDecl
@@ -113,3 +116,31 @@ class ShiftedPreNormBlock:
         if len(self.norms) == 1:
             return x
         return self.feed_forward.forward(self.norms[1].forward(x), x, ctx)
+
+
+ROUNDED = "rounded stream"       # StepContext.shared: (the stream's tensor, its values in the engine dtype)
+
+
+@register_arrangement("post_norm")
+class PostNormBlock:
+    leaves_rounded = True        # forward() leaves ctx.shared[ROUNDED] in step with the stream it returns
+
+    def __init__(self, spec, norms, mixer, feed_forward):
+        if len(norms) not in (1, 2):
+            raise ValueError(f"a post-norm block takes one norm (no feed-forward) or two, got {len(norms)}")
+        if any(not hasattr(n, "add_normed") for n in norms):
+            raise ValueError("the norms of a post-norm block must offer add_normed (the RMS norm does)")
+        if hasattr(mixer, "forward_mixes"):
+            raise ValueError("a mixer that reads blends with the token before needs a norm in front of it that makes them")
+        self.spec, self.norms, self.mixer, self.feed_forward = spec, list(norms), mixer, feed_forward
+
+    def forward(self, x, ctx, cache, position):
+        known, y = ctx.shared.get(ROUNDED, (None, None))
+        if known is not x:
+            y = kernels.round_rows(x, self.norms[0].runtime.dtype)
+        factor = self.spec.residual_factor
+        y = self.norms[0].add_normed(x, self.mixer.forward_terms(y, ctx, cache, position), factor)
+        if len(self.norms) == 2:
+            y = self.norms[1].add_normed(x, self.feed_forward.forward_terms(y, ctx), factor)
+        ctx.shared[ROUNDED] = (x, y)
+        return x

@@ -107,4 +107,4 @@ class GatedDelta(Mixer):
         o = kernels.delta_rule(q, k, v, decay, beta, ctx.entry_start, ctx.entry_slot, cache.state, s.n_heads, s.n_kv_heads,
                                s.head_dim, s.value_dim)
         mixed = kernels.delta_finish(o, gate, self.out_norm, s.n_heads, s.norm_eps, proj.dtype)
-        return linear(self.runtime, mixed, self.out_w, residual=residual, out_dtype=residual.dtype, out=residual)
+        return linear(self.runtime, mixed, self.out_w, residual=residual, out_dtype=torch.float32, out=residual)

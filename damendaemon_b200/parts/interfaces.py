@@ -15,7 +15,9 @@
 Embedding         tensor_decls(spec); forward(ctx, position) -> float32 residual stream [N,width]
 Head              tensor_decls(spec); forward(x, ctx) -> float32 logits [ctx.n_wanted, vocab] at rows ctx.want_rows
 Norm              tensor_decls(spec); forward(x_f32 [N,width], row_index=None) -> [N,width] engine dtype;
-                  scale_output(factor): everything it returns is multiplied by factor from then on
+                  scale_output(factor): everything it returns is multiplied by factor from then on;
+                  optionally add_normed(x, terms, factor, rounded): x += factor * norm(the terms), in place, and x
+                  rounded to the engine dtype if asked
 PositionEncoding  tensor_decls(spec); embedding_table() -> table or None (added to the token
                   embedding by the fused embedding kernel); on_embedding(x, ctx) -> x for
                   encodings that act there without a table; on_query_key(q, k, ctx) -> (q, k)
@@ -32,7 +34,10 @@ Arrangement       cls(layer_spec, norms, mixer, feed_forward), norms being the b
                   order; forward(x, ctx, cache, position) -> x
 
 ``residual`` is the float32 residual stream; a part returns the updated stream and may
-write it in place (the GEMM epilogues add into it).
+write it in place (the GEMM epilogues add into it). ``residual`` None: the part returns its bare
+result, float32. ``forward_terms(y, ctx[, cache, position])`` of a mixer or feed-forward is its bare
+result as operands of ``kernels.post_norm`` (a tensor; or two with factors; or rows and which of them a
+token adds up), so that whatever norms and adds the result does not need it made first.
 """
 from __future__ import annotations
 
@@ -72,12 +77,18 @@ class Mixer(Part):
     def forward(self, y, residual, ctx, cache, position):
         raise NotImplementedError
 
+    def forward_terms(self, y, ctx, cache, position):
+        return {"a": self.forward(y, None, ctx, cache, position)}
+
 
 class FeedForward(Part):
     graph_safe = False
 
     def forward(self, y, residual, ctx):
         raise NotImplementedError
+
+    def forward_terms(self, y, ctx):
+        return {"a": self.forward(y, None, ctx)}
 
 
 class Norm(Part):

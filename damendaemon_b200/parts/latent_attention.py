@@ -127,4 +127,4 @@ class LatentAttention(Mixer):
                                            window=s.window, gate=gate, n_splits=ctx.key_splits(s.n_heads), kv_heads=1,
                                            v_dim=s.rank, sink=self.sink, values_in_keys=True)
         attended = kernels.per_head_linear(mixed, self.value_up, s.rank)
-        return linear(self.runtime, attended, self.out_w, residual=residual, out_dtype=residual.dtype, out=residual)
+        return linear(self.runtime, attended, self.out_w, residual=residual, out_dtype=torch.float32, out=residual)

@@ -34,12 +34,12 @@ def grouped_tile(tensor_cores, pairs, groups):
     return next((t for t in kernels.GROUPED_TCGEN05_TILES if t >= want), kernels.GROUPED_TCGEN05_TILES[-1])
 
 
-def grouped_linear(tensor_cores, a, w, tile_group, tile, out_dtype=None):
+def grouped_linear(tensor_cores, a, w, tile_group, tile, out_dtype=None, activation=None, row_scale=None):
     """Rows of a in tiles of ``tile``; tile i is multiplied with w[tile_group[i]] (w: [groups, out, in]); tiles whose
-    group is negative are skipped."""
+    group is negative are skipped. act(row_scale[r] * product), row_scale float32 [rows] or None, in the product's epilogue."""
     if tensor_cores:
-        return kernels.gemm_grouped_tcgen05(a, w, tile_group, tile, out_dtype=out_dtype or a.dtype)
-    return kernels.gemm_simt_grouped(a, w, tile_group, out_dtype=out_dtype or a.dtype)
+        return kernels.gemm_grouped_tcgen05(a, w, tile_group, tile, out_dtype=out_dtype or a.dtype, activation=activation, row_scale=row_scale)
+    return kernels.gemm_simt_grouped(a, w, tile_group, activation=activation, out_dtype=out_dtype or a.dtype, row_scale=row_scale)
 
 
 def grouped_gated_unit(tensor_cores, a, gate_up, tile_group, tile, limit, alpha, form="clamped_swish"):

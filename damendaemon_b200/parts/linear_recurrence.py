@@ -78,4 +78,4 @@ class LinearRecurrence(Mixer):
             kernels.conv_state_update(u_in, conv_state, ctx.entry_start, ctx.entry_slot)
         fade, drive = kernels.recurrence_gates(u, self.wa, self.ba, self.wi, self.bi, self.lam, s.gain)      # fade = 1 - a
         mixed = kernels.linear_scan(fade, drive, gate, ctx.entry_start, ctx.entry_slot, cache.state, activation="gelu_tanh")
-        return linear(self.runtime, mixed, self.out_w, residual=residual, out_dtype=residual.dtype, out=residual)
+        return linear(self.runtime, mixed, self.out_w, residual=residual, out_dtype=torch.float32, out=residual)

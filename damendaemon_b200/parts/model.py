@@ -4,7 +4,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels
-from . import (attention, block, delta_rule, embedding, feed_forward, head, latent_attention, linear_recurrence, norms,  # noqa: F401
+from . import (attention, block, delta_rule, embedding, feed_forward, head, latent_attention, linear_recurrence, matrix_memory, norms,  # noqa: F401
                positions, retention, side_by_side, state_space, time_mix)  # noqa: F401  (register the built-in parts)
 from .spec import TensorDecl
 from .registry import ARRANGEMENTS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSITIONS, lookup
@@ -111,7 +111,10 @@ class DecoderModel:
                 if entry.add_embedding or entry.add_vector is not None:
                     kernels.add_rows(x, first if entry.add_embedding else None,
                                      None if entry.add_vector is None else self.pass_vectors[entry.add_vector])
+                    ctx.shared.pop(block.ROUNDED, None)               # a rounded copy of the stream is no longer its copy
                 x = self.blocks[entry.layer].forward(x, ctx, caches[stop], self.position)
+                if not getattr(self.blocks[entry.layer], "leaves_rounded", False):
+                    ctx.shared.pop(block.ROUNDED, None)
         if ctx.n_wanted == 0:
             return None
         return self.head.forward(x, ctx)

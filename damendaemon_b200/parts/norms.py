@@ -54,6 +54,18 @@ class RmsNorm(Norm):
         """Multiply everything the norm returns (folded into the weight, which then is the factor itself)."""
         self.weight, self.offset = (self.offset + self.weight) * factor, 0.0
 
+    def add_normed(self, x, terms, factor=1.0, rounded=True):
+        """x += factor * norm(y) in place, y given as a sublayer's ``forward_terms``; returns x in the engine dtype (x itself
+        in a float32 engine), or None where that is not asked for. One pass over the stream."""
+        if self.spec.groups != 1:
+            raise ValueError("a result that is normed and added is normed whole, not in groups")
+        if self.offset:
+            self.weight, self.offset = self.offset + self.weight, 0.0
+        low = rounded and self.runtime.dtype != x.dtype
+        out = kernels.post_norm(x, weight=self.weight, eps=self.spec.eps, factor=factor,
+                                rounded_dtype=self.runtime.dtype if low else None, **terms)
+        return out if low or not rounded else x
+
     def forward_pair(self, other, x):
         """This norm's and another RMS norm's rows of the same x, in one pass over it."""
         y, z, _ = kernels.token_mix(x, self.weight, self.spec.eps, self.runtime.dtype, offset=self.offset, weight2=other.weight)

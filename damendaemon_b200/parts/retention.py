@@ -68,4 +68,4 @@ class Retention(Mixer):
                               s.head_dim, s.value_dim, freqs=None if self.rotary is None else self.rotary.freqs,
                               interleaved=True if self.rotary is None else self.rotary.spec.interleaved)
         mixed = kernels.retention_finish(o, gate, s.n_heads, s.norm_eps, proj.dtype)
-        return linear(self.runtime, mixed, self.out_w, residual=residual, out_dtype=residual.dtype, out=residual)
+        return linear(self.runtime, mixed, self.out_w, residual=residual, out_dtype=torch.float32, out=residual)

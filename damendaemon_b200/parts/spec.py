@@ -317,17 +317,54 @@ class LinearRecurrenceSpec:
 
 
 @dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Linear attention over a matrix memory per head that fades by one number per head and token. q = W_q y, k = W_k y
+    ([n_heads, head_dim]), v = W_v y ([n_heads, value_dim]), each through ``activation`` (None or 'silu'), q times
+    ``query_scale``; per head S <- (1 - fade) S + take k v^T, o = S^T q, S float32 per request from zero. Either ``decay`` gives
+    fade = 1 - decay per head and take = 1; or exponential gates do: i = cap tanh((W_input y + b) / cap), f = log sigmoid(cap
+    tanh((W_forget y + b) / cap)) per head, cap = ``gate_cap``, M' = max(f + M, i) from M = 0, 1 - fade = exp(f + M - M'), take =
+    exp(i - M'), and with n <- (1 - fade) n + take k the read-out is o / (max(|n . q|, exp(-M')) + ``denominator_eps``). o is
+    divided by its root mean square (``norm_eps``) per head, or (``norm_together``) over all heads at once, multiplied by
+    ``out_norm`` [n_heads * value_dim] and by sigmoid(W_gate y), and projected by W_out."""
+    kind: str            # 'matrix_memory'
+    width: int
+    n_heads: int
+    head_dim: int
+    value_dim: int
+    norm_eps: float
+    query_weight: str    # checkpoint names; matrices [out, in]
+    key_weight: str
+    value_weight: str
+    gate_weight: str
+    out_norm: str
+    out_weight: str
+    query_scale: float = 1.0
+    activation: Optional[str] = None
+    norm_together: bool = False
+    decay: Optional[Tuple[float, ...]] = None      # one per head
+    input_gate: Optional[str] = None               # [n_heads, width] and [n_heads]
+    input_gate_bias: Optional[str] = None
+    forget_gate: Optional[str] = None
+    forget_gate_bias: Optional[str] = None
+    gate_cap: float = 1.0
+    denominator_eps: float = 0.0
+
+
+@dataclass(frozen=True)
 class SideBySideSpec:
     """Two mixers that read the same input; the result is ``factor`` * (norm(left) * left_norm + norm(right) * right_norm),
-    each output divided by its root mean square over the model width (``norm_eps``) and multiplied by its weight [width]."""
+    each output divided by its root mean square over the model width (``norm_eps``) and multiplied by its weight [width].
+    Without norms (both None): ``left_scale`` * left + ``right_scale`` * right."""
     kind: str            # 'side_by_side'
     width: int
     left: object         # mixer specs
     right: object
-    left_norm: str       # checkpoint names
-    right_norm: str
-    norm_eps: float
+    left_norm: Optional[str] = None      # checkpoint names
+    right_norm: Optional[str] = None
+    norm_eps: float = 0.0
     factor: float = 0.5
+    left_scale: float = 1.0
+    right_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -357,6 +394,15 @@ class GatedUnitSpec:
     down_weight: str
     alpha: float = 1.702
     activation: str = "clamped_swish"
+
+
+@dataclass(frozen=True)
+class PlainUnitSpec:
+    """A small feed-forward of two matrices, W_down act(W_up y), no biases; ``activation`` one of the dense feed-forward's."""
+    inner: int
+    up_weight: str
+    down_weight: str
+    activation: str
 
 
 @dataclass(frozen=True)
@@ -390,12 +436,14 @@ class ScoreRoutedExpertsSpec:
     weighted by s * weight_scale, or, with ``renormalize``, by s over the sum of the chosen s (+ 1e-20). ``correction`` (a
     checkpoint name, one number per router output) is added to the scores for the choice only. The router's last ``identity``
     outputs are experts without tensors, whose output is y itself. ``shared``: a unit that runs for every token; with
-    ``shared_gate`` (a checkpoint name, [1, width]) its output is multiplied by sigmoid(gate . y)."""
+    ``shared_gate`` (a checkpoint name, [1, width]) its output is multiplied by sigmoid(gate . y). ``weight_input``: a chosen
+    expert's weight multiplies its input instead of its output, unit(weight * y); for plain units, which are the experts of a
+    layer all alike or none."""
     kind: str            # 'experts_by_score'
     width: int
     top: int
     router: str          # checkpoint name of W_router [experts + identity, width]
-    experts: Tuple[GatedUnitSpec, ...]       # all of one size and activation
+    experts: Tuple[object, ...]              # GatedUnitSpec or PlainUnitSpec, all of one size and activation
     groups: int = 1
     keep_groups: int = 1
     weight_scale: float = 1.0
@@ -405,6 +453,7 @@ class ScoreRoutedExpertsSpec:
     correction: Optional[str] = None
     renormalize: bool = False
     identity: int = 0
+    weight_input: bool = False
 
 
 @dataclass(frozen=True)
@@ -419,12 +468,14 @@ class LayerSpec:
     feed-forward; 'parallel' one norm whose output both the mixer and the feed-forward read, or two norms of the same input,
     the first for the mixer, the second for the feed-forward; 'pre_norm_shift' is
     'pre_norm', or 'pre_norm_mixer' with one norm, whose mixer reads its normed input blended per channel with the
-    normed input of the token before: n[t] + (n[t-1] - n[t]) * ``shift_weight`` [width], n[-1] = 0)."""
+    normed input of the token before: n[t] + (n[t-1] - n[t]) * ``shift_weight`` [width], n[-1] = 0; 'post_norm' norms what the
+    mixer (and, with two norms, the feed-forward) returns and adds it times ``residual_factor``)."""
     arrangement: str
     mixer: object
     feed_forward: object
     norms: Tuple[object, ...]
     shift_weight: Optional[str] = None
+    residual_factor: float = 1.0
 
     @property
     def kind(self):

@@ -84,4 +84,4 @@ class StateSpace(Mixer):
         read = kernels.state_space_scan(xbc, dt, self.dt_bias, self.decay_log, self.skip, ctx.entry_start, ctx.entry_slot, cache.state,
                                         s.n_heads, s.groups, s.state, s.value_dim)
         mixed = kernels.gated_group_norm(read, z, self.out_norm, s.norm_groups, s.norm_eps, proj.dtype)
-        return linear(self.runtime, mixed, self.out_w, residual=residual, out_dtype=residual.dtype, out=residual)
+        return linear(self.runtime, mixed, self.out_w, residual=residual, out_dtype=torch.float32, out=residual)

@@ -99,4 +99,4 @@ class TimeMix(Mixer):
             operands = kernels.time_prepare(r, k, v, decay_in, self.decay_bias, self.bonus, s.n_heads, s.head_dim, s.head_dim)
             read = kernels.time_scan(*operands, ctx.entry_start, ctx.entry_slot, cache.state, s.n_heads, s.head_dim, s.head_dim)
             mixed = kernels.retention_finish(read, gate, s.n_heads, s.norm_eps, r.dtype, weight=self.out_norm)
-        return linear(rt, mixed, self.out_w, residual=residual, out_dtype=residual.dtype, out=residual)
+        return linear(rt, mixed, self.out_w, residual=residual, out_dtype=torch.float32, out=residual)

@@ -59,4 +59,4 @@ def load_config(model_dir):
 
 
 def _load_builtin():
-    from .architectures import bonatar, derusun, godotar, gpt2, tetitar, zokanex  # noqa: F401  (register themselves on import)
+    from .architectures import bonatar, derusun, dozetar, godotar, gpt2, tetitar, zokanex  # noqa: F401  (register themselves on import)
