@@ -52,7 +52,7 @@ def _mixer_spec(c: DozetarConfig, i: int):
                          out_weight=p + "left.o", out_bias=p + "left.o.b", value_dim=l.vdim,
                          rotary=RotarySpec("rotary", head_dim=l.dim, dims=l.rot.dims, base=l.rot.base, interleaved=True),
                          query_norm=p + "left.q.norm", key_norm=p + "left.k.norm", head_norm_eps=c.norm_eps,
-                         norm_whole_projection=True, sink=p + "left.sink")
+                         norm_whole_projection=True, sink=p + "left.sink", exact_weights=True)
     right = _memory(c, m.right, p + "right.", activation="silu", norm_together=True, decay=m.right.decay)
     return SideBySideSpec("side_by_side", width=c.width, left=left, right=right, left_scale=m.left_scale, right_scale=m.right_scale)
 

@@ -5,8 +5,9 @@
 // per query row, so earlier portions of the prompt are read exactly like this step's tokens.
 // Scores, softmax and the weighted value sum are float32 (damendaemon/kernels.py:147-178 for the
 // mask and the stable softmax; damendaemon/qwen2.py:754-770 for the offset-aware causal rule).
-// Takes head sizes 64 and 128 with any number of heads and key/value groups; the general
-// kernel (attention_rows.cu) serves every other size and is its reference in the tests.
+// Takes head sizes 64 and 128 with any number of heads and key/value groups, and (dd_attention_prefill_padded) every
+// other pair of key and value head sizes that are multiples of 8 up to 128, in tiles of 64 or 128 columns whose rest is
+// zero; the general kernel (attention_rows.cu) serves all else and is its reference in the tests.
 #include "common.cuh"
 #include <math_constants.h>
 
@@ -43,7 +44,8 @@ template <int D> __device__ __forceinline__ uint32_t tile_off(int r, int c) {
     return (uint32_t)(r * D * 2 + ((c ^ (r & 7)) << 4));
 }
 
-template <int D>
+// D, DV: columns of a key and a value tile. PADDED: a key head has dk <= D and a value head dv <= DV elements.
+template <int D, int DV, bool PADDED>
 __global__ void __launch_bounds__(THREADS)
 attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ cache,
                          const int* __restrict__ entry_start, const int* __restrict__ entry_pos0, int n_entries,
@@ -51,13 +53,14 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                          int out_stride, int H, int KH, int P, int n_pages, int window, float scale_log2e,
                          int* __restrict__ error_flag, int chunk, const __nv_bfloat16* __restrict__ gate, int gate_stride,
                          int keep_first, float cap_log2e, float scale_over_cap, const float* __restrict__ sink,
-                         int exact_weights) {
-    constexpr int NC = D / 8;                 // 16-byte chunks per row
+                         int exact_weights, int dk_arg, int dv_arg) {
+    constexpr int NC = D / 8, NV = DV / 8;    // 16-byte chunks per row
     constexpr int KS = D / 16;                // k-steps over the head dimension
+    const int dk = PADDED ? dk_arg : D, dv = PADDED ? dv_arg : DV;
     extern __shared__ __align__(128) uint8_t smem[];
     uint8_t* sQ = smem;
     uint8_t* sK = sQ + BQ * D * 2;            // [2][BKV][D]
-    uint8_t* sV = sK + 2 * BKV * D * 2;       // [2][BKV][D]
+    uint8_t* sV = sK + 2 * BKV * D * 2;       // [2][BKV][DV]
     dd_launch_dependents();
     dd_grid_wait();
 
@@ -83,9 +86,9 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
     };
     const int kv_lo = first_seen(pos_first);
     const int* bt = block_table + (size_t)e * max_blocks;
-    const size_t head_plane = (size_t)P * D, page_stride = 2 * (size_t)KH * head_plane;
-    const __nv_bfloat16* k_base = cache + (size_t)kh * head_plane;
-    const __nv_bfloat16* v_base = k_base + (size_t)KH * head_plane;
+    const size_t page_stride = (size_t)KH * P * (dk + dv);       // a page's key plane, then its value plane
+    const __nv_bfloat16* k_base = cache + (size_t)kh * P * dk;
+    const __nv_bfloat16* v_base = cache + (size_t)KH * P * dk + (size_t)kh * P * dv;
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, t4 = lane & 3;
@@ -94,15 +97,16 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
     for (int idx = tid; idx < BQ * NC; idx += THREADS) {
         const int r = idx / NC, c = idx % NC;
         uint8_t* dst = sQ + tile_off<D>(r, c);
-        if (r < rows) cp_async16(dst, q + (size_t)(row0 + r) * q_stride + (size_t)h * D + c * 8);
+        if (r < rows && c * 8 < dk) cp_async16(dst, q + (size_t)(row0 + r) * q_stride + (size_t)h * dk + c * 8);
         else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
     }
     auto load_kv = [&](int kb, int buf) {
-        for (int idx = tid; idx < BKV * NC; idx += THREADS) {
-            const int r = idx / NC, c = idx % NC;
+        constexpr int NM = NC > NV ? NC : NV;
+        for (int idx = tid; idx < BKV * NM; idx += THREADS) {
+            const int r = idx / NM, c = idx % NM;
             const int key = kb + r;
-            uint8_t* dk = sK + buf * BKV * D * 2 + tile_off<D>(r, c);
-            uint8_t* dv = sV + buf * BKV * D * 2 + tile_off<D>(r, c);
+            uint8_t* to_k = sK + buf * BKV * D * 2 + tile_off<D>(r, c);
+            uint8_t* to_v = sV + buf * BKV * DV * 2 + tile_off<DV>(r, c);
             int page = -1;
             if ((key >= kv_lo || key < keep_first) && key <= pos_last) {
                 const int blk = key / P;
@@ -112,13 +116,15 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                     page = -1;
                 }
             }
-            if (page >= 0) {
-                const size_t off = (size_t)page * page_stride + (size_t)(key % P) * D + c * 8;
-                cp_async16(dk, k_base + off);
-                cp_async16(dv, v_base + off);
-            } else {                      // masked or missing keys must be zeros: 0 * stale NaN would spoil the sum
-                *reinterpret_cast<uint4*>(dk) = make_uint4(0, 0, 0, 0);
-                *reinterpret_cast<uint4*>(dv) = make_uint4(0, 0, 0, 0);
+            // masked or missing keys (and a tile's columns past the head) must be zeros: 0 * stale NaN would spoil the sum
+            const size_t at = (size_t)max(page, 0) * page_stride, in_page = (size_t)(key % P);
+            if (NC == NM || c < NC) {
+                if (page >= 0 && c * 8 < dk) cp_async16(to_k, k_base + at + in_page * dk + c * 8);
+                else *reinterpret_cast<uint4*>(to_k) = make_uint4(0, 0, 0, 0);
+            }
+            if (NV == NM || c < NV) {
+                if (page >= 0 && c * 8 < dv) cp_async16(to_v, v_base + at + in_page * dv + c * 8);
+                else *reinterpret_cast<uint4*>(to_v) = make_uint4(0, 0, 0, 0);
             }
         }
     };
@@ -132,9 +138,9 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
     load_kv(tile_key(0), 0);
     cp_commit();
 
-    float o[NC][4], m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
+    float o[NV][4], m[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
 #pragma unroll
-    for (int i = 0; i < NC; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    for (int i = 0; i < NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     uint32_t qf[KS][4];
     const int qpos[2] = {pos_first + warp * 16 + g, pos_first + warp * 16 + g + 8};
     int qlo[2];
@@ -155,7 +161,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
             }
         }
         const uint8_t* tk = sK + buf * BKV * D * 2;
-        const uint8_t* tv = sV + buf * BKV * D * 2;
+        const uint8_t* tv = sV + buf * BKV * DV * 2;
         // S = Q K^T for 16 query rows x 64 keys
         float s[8][4];
 #pragma unroll
@@ -208,7 +214,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
             }
         }
 #pragma unroll
-        for (int i = 0; i < NC; ++i) {
+        for (int i = 0; i < NV; ++i) {
             o[i][0] *= corr[0]; o[i][1] *= corr[0];
             o[i][2] *= corr[1]; o[i][3] *= corr[1];
         }
@@ -221,10 +227,10 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
             a[2] = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]);
             a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
-            for (int dp = 0; dp < NC / 2; ++dp) {
+            for (int dp = 0; dp < NV / 2; ++dp) {
                 uint32_t b[4];
                 const int mi = lane >> 3;
-                ldmatrix_x4_trans(smem_addr(tv + tile_off<D>(kk * 16 + (mi & 1) * 8 + (lane & 7), 2 * dp + (mi >> 1))), b);
+                ldmatrix_x4_trans(smem_addr(tv + tile_off<DV>(kk * 16 + (mi & 1) * 8 + (lane & 7), 2 * dp + (mi >> 1))), b);
                 mma_bf16(o[2 * dp], a, b[0], b[1]);
                 mma_bf16(o[2 * dp + 1], a, b[2], b[3]);
             }
@@ -236,10 +242,10 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
                 a2[2] = pack_bf16(s[2 * kk + 1][0] - bf16_low(a[2]), s[2 * kk + 1][1] - bf16_high(a[2]));
                 a2[3] = pack_bf16(s[2 * kk + 1][2] - bf16_low(a[3]), s[2 * kk + 1][3] - bf16_high(a[3]));
 #pragma unroll
-                for (int dp = 0; dp < NC / 2; ++dp) {
+                for (int dp = 0; dp < NV / 2; ++dp) {
                     uint32_t b[4];
                     const int mi = lane >> 3;
-                    ldmatrix_x4_trans(smem_addr(tv + tile_off<D>(kk * 16 + (mi & 1) * 8 + (lane & 7), 2 * dp + (mi >> 1))), b);
+                    ldmatrix_x4_trans(smem_addr(tv + tile_off<DV>(kk * 16 + (mi & 1) * 8 + (lane & 7), 2 * dp + (mi >> 1))), b);
                     mma_bf16(o[2 * dp], a2, b[0], b[1]);
                     mma_bf16(o[2 * dp + 1], a2, b[2], b[3]);
                 }
@@ -265,31 +271,31 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, cons
             inv = keep / (l[r] * keep + exp2f(s2 - m2));
         }
         if (gate) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)(row0 + row) * gate_stride + h])));
-        __nv_bfloat16* dst = out + (size_t)(row0 + row) * out_stride + (size_t)h * D + 2 * t4;
+        __nv_bfloat16* dst = out + (size_t)(row0 + row) * out_stride + (size_t)h * dv + 2 * t4;
 #pragma unroll
-        for (int i = 0; i < NC; ++i)
-            *reinterpret_cast<uint32_t*>(dst + i * 8) = pack_bf16(o[i][2 * r] * inv, o[i][2 * r + 1] * inv);
+        for (int i = 0; i < NV; ++i)
+            if (!PADDED || i * 8 < dv) *reinterpret_cast<uint32_t*>(dst + i * 8) = pack_bf16(o[i][2 * r] * inv, o[i][2 * r + 1] * inv);
     }
 }
 
-template <int D>
+template <int D, int DV, bool PADDED>
 int launch(const void* q, int q_stride, const void* cache, const int* entry_start, const int* entry_pos0, int n_entries,
            int n_tokens, const int* block_table, int max_blocks, void* out, int out_stride, int H, int KH, int P,
            int n_pages, int window, float scale, int* error_flag, cudaStream_t s, int chunk, const void* gate, int gate_stride,
-           int keep_first, float softcap, const float* sink, int exact_weights) {
-    constexpr int SMEM = (BQ + 4 * BKV) * D * 2;
+           int keep_first, float softcap, const float* sink, int exact_weights, int dk, int dv) {
+    constexpr int SMEM = ((BQ + 2 * BKV) * D + 2 * BKV * DV) * 2;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<D, DV, PADDED>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
         if (e != cudaSuccess) return dd_fail("dd_attention_prefill: shared memory refused: %s", cudaGetErrorString(e));
         configured = true;
     }
     // an upper bound of the number of 64-row tiles; blocks beyond the real count return at once
     dim3 grid(dd_ceil_div(n_tokens, BQ) + n_entries, H);
-    dd_launch(attention_prefill_kernel<D>, dim3(grid), dim3(THREADS), SMEM, s, (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)cache,
+    dd_launch(attention_prefill_kernel<D, DV, PADDED>, dim3(grid), dim3(THREADS), SMEM, s, (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)cache,
         entry_start, entry_pos0, n_entries, block_table, max_blocks, (__nv_bfloat16*)out, out_stride, H, KH, P, n_pages,
         window, scale * 1.4426950408889634f, error_flag, chunk, (const __nv_bfloat16*)gate, gate_stride, keep_first,
-        softcap * 1.4426950408889634f, softcap > 0.f ? scale / softcap : 0.f, sink, exact_weights);
+        softcap * 1.4426950408889634f, softcap > 0.f ? scale / softcap : 0.f, sink, exact_weights, dk, dv);
     return dd_check_launch("dd_attention_prefill");
 }
 }  // namespace
@@ -322,12 +328,43 @@ DD_API int dd_attention_prefill_sinks(const void* q, int q_stride, const void* c
     if (n_heads > 65535) return dd_fail("dd_attention_prefill: too many heads");
     cudaStream_t s = (cudaStream_t)stream;
     if (head_dim == 64)
-        return launch<64>(q, q_stride, cache, entry_start, entry_pos0, n_entries, n_tokens, block_table, max_blocks, out,
+        return launch<64, 64, false>(q, q_stride, cache, entry_start, entry_pos0, n_entries, n_tokens, block_table, max_blocks, out,
                           out_stride, n_heads, n_kv_heads, page_size, n_pages, window, scale, error_flag, s, chunk, gate, gate_stride,
-                          keep_first, softcap, sink, exact_weights);
-    return launch<128>(q, q_stride, cache, entry_start, entry_pos0, n_entries, n_tokens, block_table, max_blocks, out,
+                          keep_first, softcap, sink, exact_weights, 64, 64);
+    return launch<128, 128, false>(q, q_stride, cache, entry_start, entry_pos0, n_entries, n_tokens, block_table, max_blocks, out,
                        out_stride, n_heads, n_kv_heads, page_size, n_pages, window, scale, error_flag, s, chunk, gate, gate_stride,
-                       keep_first, softcap, sink, exact_weights);
+                       keep_first, softcap, sink, exact_weights, 128, 128);
+}
+
+DD_API int dd_attention_prefill_padded_supported(int n_heads, int n_kv_heads, int head_dim, int v_dim, int dtype) {
+    return dtype == DD_BF16 && n_kv_heads > 0 && n_heads % n_kv_heads == 0 && head_dim > 0 && head_dim <= 128 && head_dim % 8 == 0 &&
+           v_dim > 0 && v_dim <= 128 && v_dim % 8 == 0;
+}
+
+// dd_attention_prefill_sinks for key heads of head_dim and value heads of v_dim elements (multiples of 8 up to 128): a page
+// of the cache is its key plane [kv_heads, page_size, head_dim] followed by its value plane [kv_heads, page_size, v_dim]; out
+// has rows of n_heads * v_dim elements.
+DD_API int dd_attention_prefill_padded(const void* q, int q_stride, const void* cache, const int* entry_start,
+                                const int* entry_pos0, int n_entries, int n_tokens, const int* block_table,
+                                int max_blocks, void* out, int out_stride, int n_heads, int n_kv_heads, int head_dim,
+                                int page_size, int n_pages, int window, float scale, int* error_flag, void* stream,
+                                int chunk, const void* gate, int gate_stride, int keep_first, float softcap,
+                                const float* sink, int exact_weights, int v_dim) {
+    if (n_tokens <= 0 || n_entries <= 0) return 0;
+    if (keep_first < 0 || softcap < 0.f) return dd_fail("dd_attention_prefill: keep_first %d and softcap %g must not be negative", keep_first, softcap);
+    if (!dd_attention_prefill_padded_supported(n_heads, n_kv_heads, head_dim, v_dim, DD_BF16))
+        return dd_fail("dd_attention_prefill: needs head sizes that are multiples of 8 up to 128 and heads a multiple of key/value heads (got %d, %d, %d, %d)",
+                       n_heads, n_kv_heads, head_dim, v_dim);
+    if (q_stride % 8 || out_stride % 2 || ((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 3))
+        return dd_fail("dd_attention_prefill: rows must be 16-byte aligned");
+    if (n_heads > 65535) return dd_fail("dd_attention_prefill: too many heads");
+    cudaStream_t s = (cudaStream_t)stream;
+#define DD_PADDED(D, DV)                                                                                                              return launch<D, DV, true>(q, q_stride, cache, entry_start, entry_pos0, n_entries, n_tokens, block_table, max_blocks, out,                                  out_stride, n_heads, n_kv_heads, page_size, n_pages, window, scale, error_flag, s, chunk, gate,                                  gate_stride, keep_first, softcap, sink, exact_weights, head_dim, v_dim)
+    if (head_dim <= 64 && v_dim <= 64) DD_PADDED(64, 64);
+    if (head_dim <= 64) DD_PADDED(64, 128);
+    if (v_dim <= 64) DD_PADDED(128, 64);
+    DD_PADDED(128, 128);
+#undef DD_PADDED
 }
 
 DD_API int dd_attention_prefill(const void* q, int q_stride, const void* cache, const int* entry_start,

@@ -107,6 +107,10 @@ _SIGNATURES = {
         "dd_attention_prefill_supported": [_c_int] * 4,
         "dd_attention_prefill": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int]
                                 + [_c_int] * 6 + [_c_float, _c_void, _c_void, _c_int, _c_void, _c_int],
+        "dd_attention_prefill_padded_supported": [_c_int] * 5,
+        "dd_attention_prefill_padded": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int]
+                                       + [_c_int] * 6 + [_c_float, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_float, _c_void, _c_int,
+                                          _c_int],
         "dd_attention_prefill_sinks": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int]
                                       + [_c_int] * 6 + [_c_float, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_float, _c_void, _c_int],
         "dd_attention_latent_supported": [_c_int] * 3,
@@ -1524,6 +1528,34 @@ def attention_decode(q, cache, token_entry, positions, block_table, n_heads, sca
 
 def attention_prefill_supported(n_heads, kv_heads, head_dim, dtype):
     return dtype == torch.bfloat16 and bool(library("tensor").dd_attention_prefill_supported(n_heads, kv_heads, head_dim, BF16))
+
+
+def attention_prefill_padded_supported(n_heads, kv_heads, head_dim, v_dim, dtype):
+    return dtype == torch.bfloat16 and bool(
+        library("tensor").dd_attention_prefill_padded_supported(n_heads, kv_heads, head_dim, v_dim, BF16))
+
+
+def attention_prefill_padded(q, cache, entry_start, entry_pos0, block_table, n_heads, scale, window=None, out=None, chunk=None,
+                             gate=None, keep_first=0, softcap=None, sink=None, exact_weights=False, kv_heads=None, v_dim=None):
+    """``attention_prefill``'s kernel 'mma' for head sizes it does not take as they are (multiples of 8 up to 128, also a value
+    head of another size than a key head): its tiles' columns past the heads are zeros. cache, kv_heads, v_dim: as
+    ``attention_rows``."""
+    n, n_entries, head_dim = q.shape[0], entry_pos0.numel(), q.shape[1] // n_heads
+    n_pages, kv_heads, page_size, head_dim, v_dim = cache_geometry(cache, kv_heads, head_dim, v_dim)
+    if sink is not None and (sink.numel() != n_heads or sink.dtype != torch.float32 or not sink.is_contiguous()):
+        raise KernelError("attention: the sink must be float32 [heads]")
+    if q.shape[1] != n_heads * head_dim or q.stride(1) != 1 or q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 \
+            or not cache.is_contiguous() or entry_start.numel() != n_entries + 1:
+        raise KernelError("attention_prefill: q or the entry arrays do not fit the cache")
+    if out is None:
+        out = torch.empty((n, n_heads * v_dim), dtype=q.dtype, device=q.device)
+    _call(library("tensor"), "dd_attention_prefill_padded", _ptr(q, "q"), q.stride(0), _ptr(cache, "cache"),
+          _ptr(entry_start, "entry_start", torch.int32), _ptr(entry_pos0, "entry_pos0", torch.int32), n_entries, n,
+          _ptr(block_table, "block_table", torch.int32), block_table.shape[1], _ptr(out, "out"), out.stride(0),
+          n_heads, kv_heads, head_dim, page_size, n_pages, 0 if window is None else int(window), float(scale),
+          _ptr(error_flag(q.device)), _stream(), *_gate_args(gate, q, n_heads, chunk), int(keep_first or 0), float(softcap or 0.0),
+          _ptr(sink, "sink"), int(bool(exact_weights)), v_dim)
+    return out
 
 
 def attention_prefill_tcgen05_supported(n_heads, kv_heads, head_dim, page_size, dtype):

@@ -1,7 +1,8 @@
 """Paged causal attention of a step's tokens: the cache write and the choice of kernel.
 
 Five kernels can serve (csrc/attention_*.cu): the general one (any sizes, both dtypes: the float32 path, the
-fallback and the reference of the others), two bfloat16 decode kernels (rows by cp.async; whole pages of a group of
+fallback and the reference of the others; the mma.sync prompt kernel takes the portions of other head sizes in padded
+tiles), two bfloat16 decode kernels (rows by cp.async; whole pages of a group of
 heads by TMA) and two bfloat16 prompt kernels (mma.sync; tcgen05). Which one a step takes depends on the step
 (decode only or not, how many (token, head) pairs), on what each kernel supports (head size, page size, groups) and
 on thresholds that were measured, which are data: ``AttentionTuning``, a field of the runtime, not constants of a
@@ -65,13 +66,12 @@ def paged_attention(ctx, q, k, v, cache, n_heads, scale, window=None, chunk=None
     exact = dict(more, exact_weights=exact_weights) if special else {}
     if value_dim is not None and value_dim != cache.group.need.head_dim:
         need = cache.group.need
-        # value heads of their own size: the general kernel, which is told the page's geometry
+        # value heads of their own size: kernels that are told the page's geometry
         if cache.writable:
             kernels.kv_store(k, v, ctx.token_entry, ctx.positions, table, kv, kv_heads=need.kv_heads, head_dim=need.head_dim,
                              v_dim=value_dim)
-        return kernels.attention_rows(q, kv, ctx.token_entry, ctx.positions, table, n_heads, scale, window,
-                                      n_splits=ctx.key_splits(n_heads), chunk=chunk, gate=gate, kv_heads=need.kv_heads,
-                                      v_dim=value_dim, **more)
+        return general_attention(ctx, q, kv, table, n_heads, scale, window, need.kv_heads, need.head_dim, value_dim, exact_weights,
+                                 chunk=chunk, gate=gate, **more)
     kv_heads, page_size, head_dim = kv.shape[2], kv.shape[3], kv.shape[4]
     k_new, v_new = (k, v) if cache.writable else (None, None)
     fast = runtime.attention != "rows"
@@ -132,5 +132,27 @@ def paged_attention(ctx, q, k, v, cache, n_heads, scale, window=None, chunk=None
     if mma:
         return kernels.attention_prefill(q, kv, ctx.entry_start[n1:], ctx.entry_pos0[n1:], table[n1:], n_heads, scale, window,
                                          out=out, **masked, **exact)
-    return kernels.attention_rows(q, kv, ctx.token_entry, ctx.positions, table, n_heads, scale, window,
-                                  n_splits=ctx.key_splits(n_heads), chunk=chunk, gate=gate, **(more if special else {}))
+    return general_attention(ctx, q, kv, table, n_heads, scale, window, kv_heads, head_dim, head_dim, exact_weights, chunk=chunk,
+                             gate=gate, **(more if special else {}))
+
+
+def general_attention(ctx, q, kv, table, n_heads, scale, window, kv_heads, head_dim, value_dim, exact_weights=False, gate=None, **mask):
+    """Head sizes that have no kernel of their own, the keys and values in the cache already: the general kernel; for a step with
+    portions in bfloat16 its single tokens only (cut into splits of the keys), the portions on the tensor cores in tiles padded
+    to the next size, where the sizes allow it."""
+    runtime = ctx.runtime
+    sizes = {} if value_dim == head_dim else dict(kv_heads=kv_heads, v_dim=value_dim)
+    if ctx.decode_only or runtime.attention == "rows" or \
+            not kernels.attention_prefill_padded_supported(n_heads, kv_heads, head_dim, value_dim, q.dtype):
+        return kernels.attention_rows(q, kv, ctx.token_entry, ctx.positions, table, n_heads, scale, window,
+                                      n_splits=ctx.key_splits(n_heads), gate=gate, **mask, **sizes)
+    import torch
+    out = torch.empty((q.shape[0], n_heads * value_dim), dtype=q.dtype, device=q.device)
+    n1 = ctx.n_single
+    if n1:
+        kernels.attention_rows(q[:n1], kv, ctx.token_entry[:n1], ctx.positions[:n1], table, n_heads, scale, window, out=out[:n1],
+                               n_splits=ctx.key_splits(n_heads, n_tokens=n1), gate=None if gate is None else gate[:n1], **mask, **sizes)
+    if n1 < ctx.n_entries:
+        kernels.attention_prefill_padded(q, kv, ctx.entry_start[n1:], ctx.entry_pos0[n1:], table[n1:], n_heads, scale, window, out=out,
+                                         gate=gate, exact_weights=exact_weights, **mask, **sizes)
+    return out

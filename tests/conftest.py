@@ -50,7 +50,8 @@ TINY_E = {
     "layer_norm_epsilon": 1e-5, "activation_function": "gelu",
     "scale_attn_by_inverse_layer_idx": False,
 }
-# head size 80 (a step of 16 that no tensor-core attention kernel takes): the general kernel in both dtypes; seven heads
+# head size 80 (a step of 16 that no attention kernel takes as it is): padded tiles for prompts, the general kernel for single
+# tokens and in float32; seven heads
 TINY_F = {
     "architectures": ["GPT2LMHeadModel"], "model_type": "gpt2",
     "n_layer": 1, "n_embd": 560, "n_head": 7, "n_inner": 600, "vocab_size": 257, "n_positions": 80,

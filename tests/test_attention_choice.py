@@ -14,8 +14,9 @@ class Recorder:
     """The functions of the kernels module that paged_attention calls; every call is noted, nothing runs."""
     ATTENTION_PREFILL_TCGEN05_KEY_BLOCK = 128
 
-    def __init__(self, head_dims_decode=(64, 128), tcgen05=True, mma=True, pages=True):
+    def __init__(self, head_dims_decode=(64, 128), tcgen05=True, mma=True, pages=True, padded=False):
         self.calls = []
+        self.padded = padded
         self.head_dims_decode, self.tcgen05, self.mma, self.pages = head_dims_decode, tcgen05, mma, pages
 
     def attention_decode_supported(self, n_heads, kv_heads, head_dim, dtype):
@@ -29,6 +30,14 @@ class Recorder:
 
     def attention_prefill_supported(self, n_heads, kv_heads, head_dim, dtype):
         return self.mma and dtype == torch.bfloat16
+
+    def attention_prefill_padded_supported(self, n_heads, kv_heads, head_dim, v_dim, dtype):
+        return self.padded and dtype == torch.bfloat16
+
+    def attention_prefill_padded(self, q, kv, entry_start, entry_pos0, table, n_heads, scale, window=None, out=None, chunk=None,
+                                 gate=None, keep_first=0, softcap=None, sink=None, exact_weights=False, kv_heads=None, v_dim=None):
+        self.calls.append(("prefill-padded", entry_pos0.numel(), table.shape[0], exact_weights))
+        return out
 
     def attention_decode_pages_splits(self, n_tokens, n_heads, page_size, context, device):
         return 4
@@ -46,7 +55,7 @@ class Recorder:
         return out if out is not None else q
 
     def attention_rows(self, q, kv, token_entry, positions, table, n_heads, scale, window=None, n_splits=1, out=None,
-                       chunk=None, gate=None, kv_heads=None, v_dim=None):
+                       chunk=None, gate=None, kv_heads=None, v_dim=None, keep_first=0, softcap=None, sink=None):
         self.calls.append(("rows", q.shape[0], n_splits))
         return q
 
@@ -145,3 +154,22 @@ def test_a_sink_alone_still_takes_the_tcgen05_prompt_kernel(recorder):
     ctx, q, k, v, cache = step(8, [])
     pa.paged_attention(ctx, q, k, v, cache, 25, 0.125, window=100, sink=sink)
     assert recorder.calls == [("decode-rows+sink", 8, True, True)]          # the page-streaming kernel takes no sink
+
+
+def test_portions_of_other_head_sizes_take_the_padded_prompt_kernel(monkeypatch):
+    """Head sizes without a kernel of their own: single tokens of a mixed step go to the general kernel (with splits of the
+    keys), portions to the padded prompt kernel; a decode step, and an engine told to use rows, to the general kernel alone."""
+    r = Recorder(head_dims_decode=(), tcgen05=False, mma=False, padded=True)
+    monkeypatch.setattr(pa, "kernels", r)
+    ctx, q, k, v, cache = step(2, [40, 3], heads=4, head_dim=40)
+    pa.paged_attention(ctx, q, k, v, cache, 4, 0.1, window=9, keep_first=2, exact_weights=True)
+    assert r.calls[:1] == [("kv_store", 45)] and r.calls[2:] == [("prefill-padded", 2, 2, True)]
+    assert r.calls[1][:2] == ("rows", 2) and r.calls[1][2] > 1
+    r.calls.clear()
+    ctx, q, k, v, cache = step(5, [], heads=4, head_dim=40)
+    pa.paged_attention(ctx, q, k, v, cache, 4, 0.1)
+    assert [c[:2] for c in r.calls] == [("kv_store", 5), ("rows", 5)]
+    r.calls.clear()
+    ctx, q, k, v, cache = step(0, [20], heads=4, head_dim=40, attention="rows")
+    pa.paged_attention(ctx, q, k, v, cache, 4, 0.1)
+    assert r.calls == [("kv_store", 20), ("rows", 20, 1)]
