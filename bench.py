@@ -384,6 +384,21 @@ GODOTAR_KERNEL_PAIRS = [     # (a kernel of Godotar, the like kernel of the clos
     ("perheadturn_m2048", "perhead_m2048"), ("perheadturn_m8", "perhead_m8"),
     ("grouped_softmax_m2048", "grouped_score_m2048"), ("grouped_softmax_m8", "grouped_score_m8"),
 ]
+DOZETAR_KERNEL_PAIRS = [     # (a kernel of Dozetar, the like kernel of the closest models: Godotar and Zokanex, for kept first keys Derusun) at width 1600
+    ("postnorm_m2048", "rmsnorm_m2048"), ("postnorm_m8", "rmsnorm_m8"), ("postnormpair_m2048", "pairnorm_m2048"), ("postnormpair_m8", "pairnorm_m8"),
+    ("memgates_p2_t1024", None), ("memgates_p8_t1", None),
+    ("memprep_p2_t1024", "timeprep_p2_t1024"), ("memscan_p2_t1024", "timescan_p2_t1024"), ("memfinish_p2_t1024", "timefinish_p2_t1024"),
+    ("memstep_p8_t1", "timestep_p8_t1"), ("memstep_p64_t1", "timestep_p64_t1"),
+    ("memscan_p2_t1024_k256v512", "timescan_p2_t1024"), ("memstep_p8_t1_k256v512", "timestep_p8_t1"), ("memstep_p64_t1_k256v512", "timestep_p64_t1"),
+    ("memdecayprep_p2_t1024", "timeprep_p2_t1024"), ("memdecayscan_p2_t1024", "retention_p2_t1024"), ("memdecayfinish_p2_t1024", "retfinish_p2_t1024"),
+    ("memdecaystep_p8_t1", "retention_p8_t1"), ("memdecaystep_p64_t1", "retention_p64_t1"), ("memdecayfinish_p8_t1", "retfinish_p8_t1"),
+    ("widenorm_m2048", "headnorm_m2048"), ("widenorm_m8", "headnorm_m8"),
+    ("sinks_prefill_p2_t1024", "sinks_prefill_p2_t1024"), ("sinks_decode_b8_c768", "sinks_decode_b8_c768"),
+    ("padded_prefill_p2_t1024", "sinks_prefill_p2_t1024"), ("padded_decode_b8_c768", "sinks_decoderows_b8_c768"),
+    ("padded_decode_b64_c768", "sinks_decoderows_b64_c768"),
+    ("grouped_upplain_m2048", "grouped_upsilu_m2048"), ("grouped_upplain_m8", "grouped_upsilu_m8"),
+    ("grouped_plainscore_m2048", "grouped_score_m2048"), ("grouped_plainscore_m8", "grouped_score_m8"),
+]
 CUDA_CORE_FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12      # nominal: 148 SMs x 128 lanes x one fused multiply-add a cycle at 1,965 MHz
 
 
@@ -498,6 +513,34 @@ def godotar_configs(size, layers, vocab=50257):
     return out
 
 
+def dozetar_configs(size, layers, vocab=50257):
+    """Godotar (layers of time mixing; its looped mix with experts), Zokanex (retention layers; its mix with experts) and Dozetar
+    models whose layers have one size: matrix memories alone; parallel layers alone; and memories and parallel layers in turn (a
+    parallel layer as every third); each with experts of Zokanex's sizes in every layer, and the last also with value heads of 48
+    and key heads of 96 (whole tiles padded)."""
+    z = DESIGN_SIZES[size]
+    out = {k: v for k, v in godotar_configs(size, layers, vocab).items() if k in ("godotar_wkv_dense", "godotar_looped_experts")}
+    out.update({k: v for k, v in zokanex_configs(size, layers, vocab).items() if k in ("zokanex_retention_dense", "zokanex_mixed_experts")})
+    heads = z["heads"]
+    memory = {"heads": heads, "dim": 64, "vdim": 64, "gate_cap": 12.0}
+    decay = [1.0 - 2.0 ** -(1 + 9 * h / max(1, heads - 1)) for h in range(heads)]
+
+    def parallel(dim, vdim):
+        left = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "rot": {"dims": dim // 2, "base": 10000.0},
+                "mask": {"size": 1024, "keep_first": 4}}
+        return {"left": left, "right": {"heads": heads, "dim": 64, "vdim": 64, "decay": decay}, "left_scale": 0.6, "right_scale": 0.5}
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["expert_ff"]}}
+
+    def model(entries):
+        return {"architecture": "Dozetar", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+                "logit_softcap": 30.0, "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in entries]}
+    out["dozetar_memory_experts"] = model([("mlstm", memory)] * layers)
+    out["dozetar_parallel_experts"] = model([("parallel", parallel(64, 64))] * layers)
+    out["dozetar_mixed_experts"] = model([("parallel", parallel(64, 64)) if i % 3 == 1 else ("mlstm", memory) for i in range(layers)])
+    out["dozetar_mixed_96_48_experts"] = model([("parallel", parallel(96, 48)) if i % 3 == 1 else ("mlstm", memory) for i in range(layers)])
+    return out
+
+
 def design_configs(size, layers, vocab=50257):
     """GPT-2 and two Bonatar models (dense layers only; expert layers only) whose layers have one size."""
     z = DESIGN_SIZES[size]
@@ -516,7 +559,7 @@ def design_configs(size, layers, vocab=50257):
 def design_bench(args):
     """``--design bonatar`` (beside GPT-2), ``--design zokanex`` (beside Bonatar, the closest model), ``--design derusun`` or
     ``--design tetitar`` (each beside Zokanex, the closest model), ``--design godotar`` (beside Derusun, and Zokanex for the
-    experts): prefill and decode
+    experts), ``--design dozetar`` (beside Godotar and Zokanex): prefill and decode
     throughput at equal layer sizes (random
     bfloat16 weights, a few layers), and each kernel of the new design beside the like kernel of the other, timed in a
     chain replayed from a CUDA graph over inputs that rotate through more memory than L2 holds."""
@@ -527,6 +570,7 @@ def design_bench(args):
     layers = args.layers or 6
     configs_of, pairs = {"zokanex": (zokanex_configs, ZOKANEX_KERNEL_PAIRS), "derusun": (derusun_configs, DERUSUN_KERNEL_PAIRS),
                          "tetitar": (tetitar_configs, TETITAR_KERNEL_PAIRS), "godotar": (godotar_configs, GODOTAR_KERNEL_PAIRS),
+                         "dozetar": (dozetar_configs, DOZETAR_KERNEL_PAIRS),
                          "bonatar": (design_configs, DESIGN_KERNEL_PAIRS)}[args.design]
     out = {"design": args.design, "layers": layers, "dtype": "bf16", "data": "synthetic", "peaks": dict(measured_peaks, source=peaks_from),
            "sizes": {}, "kernels": [],
@@ -610,7 +654,7 @@ def main():
     parser.add_argument("--case-iters", type=int, default=50)
     parser.add_argument("--case-graph", action="store_true", help="time the kernel case as launches replayed from one CUDA graph")
     parser.add_argument("--workload", choices=sorted(WORKLOADS), help="run a scheduler workload instead of the headline bench")
-    parser.add_argument("--design", choices=("bonatar", "zokanex", "derusun", "tetitar", "godotar"), help="another design beside GPT-2 (zokanex: beside Bonatar; derusun and tetitar: beside Zokanex; godotar: beside Derusun) at equal layer sizes (prefill, decode, "
+    parser.add_argument("--design", choices=("bonatar", "zokanex", "derusun", "tetitar", "godotar", "dozetar"), help="another design beside GPT-2 (zokanex: beside Bonatar; derusun and tetitar: beside Zokanex; godotar: beside Derusun; dozetar: beside Godotar and Zokanex) at equal layer sizes (prefill, decode, "
                         "kernel by kernel) instead of the headline bench")
     parser.add_argument("--parity", action="store_true", help="the float32 engine beside the bfloat16 one: on the benchmark's model "
                         "(logit differences, greedy agreement), or with --workload on that workload (the same requests in both)")

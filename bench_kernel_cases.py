@@ -496,6 +496,82 @@ def _time_mix_case(entries, length, dev, which):
     return run, {"bytes": entries * H * D * D * 8 + tokens * inner * 4 * 5, "flops": 6 * tokens * H * D * D, "fp32": True}
 
 
+def _memory_case(entries, length, dev, which, gated=True, dk=D, dv=D, heads=H):
+    """A matrix memory of `entries` requests of `length` tokens each in one step (25 heads of 64 by 64 unless told): 'scan' the
+    recurrence over the float32 state, 'prep' its operands, 'gates' the gates of the tokens, 'finish' the read-out's denominator,
+    norm, weight and gate, 'step' single tokens (gated: all of it in one kernel; fixed decays: the recurrence). Float32 sums on the
+    CUDA cores."""
+    tokens, ent, start, slot = _entries(entries, length, dev)
+    qk, inner = heads * dk, heads * dv
+    shape = K.memory_state_shape(heads, dk, dv, gated)
+    state_bytes = entries * shape[0] * shape[1] * shape[2] * 8
+    copies = max(2, min(24, (300 << 20) // max(1, tokens * 2 * (qk + inner) * 2 + state_bytes // 2)))
+    projs = [torch.randn(tokens, 2 * qk + 2 * inner, device=dev).mul_(0.5).to(torch.bfloat16) for _ in range(copies)]
+    split = lambda p: (p[:, :qk], p[:, qk:2 * qk], p[:, 2 * qk:2 * qk + inner], p[:, 2 * qk + inner:])
+    z, weight = torch.randn(tokens, 2 * heads, device=dev), torch.ones(inner, device=dev)
+    z[:, heads:] += 3.0
+    fade = torch.full((heads,), 0.01, device=dev)
+    states = [torch.zeros(entries, *shape, device=dev) for _ in range(copies)]
+    peak = torch.zeros(entries, heads, device=dev)
+    out = torch.empty(tokens, inner, device=dev, dtype=torch.bfloat16)
+    silu = not gated
+    if which == "step":
+        more = dict(weight=weight, eps=1e-6, den_eps=1e-6, gates=(z, 12.0, peak), out=out) if gated else dict(fade=fade, silu=True)
+        run = lambda i: K.memory_step(*split(projs[i % copies]), slot, states[i % copies], heads, dk, dv, **more)
+        return run, {"bytes": state_bytes + tokens * 2 * (2 * qk + 3 * inner), "flops": 5 * tokens * heads * shape[1] * dk, "fp32": True}
+    if which == "gates":
+        run = lambda i: K.memory_gates(z, 12.0, start, slot, peak)
+        return run, {"bytes": tokens * heads * 20, "flops": 40 * tokens * heads, "fp32": True}
+    take = torch.ones(tokens, heads, device=dev) if gated else None
+    if which == "prep":
+        run = lambda i: K.memory_prepare(*split(projs[i % copies])[:3], heads, dk, dv, silu=silu, take=take)
+        return run, {"bytes": tokens * (2 * qk + inner) * 6, "flops": 4 * tokens * (2 * qk + inner), "fp32": True}
+    if which == "finish":
+        o = torch.randn(tokens, heads, -(-(dv + (1 if gated else 0)) // 4) * 4, device=dev)
+        floor = torch.ones(tokens, heads, device=dev) if gated else None
+        run = lambda i: K.memory_finish(o, split(projs[i % copies])[3], weight, heads, dv, 1e-6, 1e-6, floor=floor, together=not gated, out=out)
+        return run, {"bytes": tokens * inner * 8, "flops": 10 * tokens * inner}
+    ops = [K.memory_prepare(*split(p)[:3], heads, dk, dv, silu=silu, take=take) for p in projs[:min(copies, 6)]]
+    fades = torch.full((tokens, heads), 0.01, device=dev) if gated else fade
+    o = torch.empty_like(ops[0][2])
+    run = lambda i: K.memory_scan(*ops[i % len(ops)], fades, start, slot, states[i % copies], dk, dv, out=o)
+    return run, {"bytes": state_bytes + tokens * (2 * qk + 2 * inner) * 4, "flops": 5 * tokens * heads * shape[1] * dk, "fp32": True}
+
+
+def _post_norm_case(rows, dev, which):
+    """A result (two results with factors; the sum of two rows a token) normed, added to the stream and rounded (width 1600)."""
+    width = H * D
+    copies = max(2, min(24, (300 << 20) // (rows * width * 14)))
+    x = [torch.randn(rows, width, device=dev) for _ in range(copies)]
+    a, b = ([torch.randn(rows * (2 if which == "rows" else 1), width, device=dev) for _ in range(copies)] for _ in range(2))
+    w = torch.ones(width, device=dev)
+    pair = torch.randperm(2 * rows, device=dev).to(torch.int32)
+    terms = {"one": lambda i: {}, "pair": lambda i: {"other": b[i], "scale": 0.6, "other_scale": 0.5}, "rows": lambda i: {"pair_row": pair}}[which]
+    run = lambda i: K.post_norm(x[i % copies], a[i % copies], w, 1e-6, 0.7, rounded_dtype=torch.bfloat16, **terms(i % copies))
+    return run, {"bytes": rows * width * (10 + (4 if which == "one" else 8)), "flops": 6 * rows * width}
+
+
+def _padded_case(batch, length, dev, decode, dk=96, dv=48, heads=H):
+    """Attention whose value heads (48) are smaller than its key heads (96), with a window that holds the whole context, kept first
+    keys and a sink: prompts in padded tiles, single tokens through the general kernel."""
+    tokens, n_pages = (batch if decode else batch * length), batch * (-(-length // PAGE))
+    copies = max(2, min(12, (300 << 20) // (batch * length * heads * (dk + dv) * 2)))
+    caches = [torch.randn(n_pages, heads * PAGE * (dk + dv), device=dev).to(torch.bfloat16) for _ in range(copies)]
+    table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(batch, -1)
+    q = torch.randn(tokens, heads * dk, device=dev).to(torch.bfloat16)
+    kw = dict(window=1024 * (-(-length // 1024)), keep_first=4, sink=torch.zeros(heads, device=dev), kv_heads=heads, v_dim=dv)
+    if decode:
+        ent = torch.arange(batch, dtype=torch.int32, device=dev)
+        pos = torch.full((batch,), length - 1, dtype=torch.int32, device=dev)
+        splits = max(1, min(-(-(K.sm_count(dev) * 16) // (batch * heads)), (length + 63) // 64, 32))
+        run = lambda i: K.attention_rows(q, caches[i % copies], ent, pos, table, heads, dk ** -0.5, n_splits=splits, **kw)
+        return run, {"bytes": batch * length * heads * (dk + dv) * 2, "flops": 2 * batch * length * heads * (dk + dv)}
+    start = torch.arange(batch + 1, dtype=torch.int32, device=dev) * length
+    pos0 = torch.zeros(batch, dtype=torch.int32, device=dev)
+    run = lambda i: K.attention_prefill_padded(q, caches[i % copies], start, pos0, table, heads, dk ** -0.5, exact_weights=True, **kw)
+    return run, {"bytes": batch * length * heads * (2 * dk + 2 * dv) * 2, "flops": batch * (length * (length + 1)) * heads * (dk + dv)}
+
+
 def _square_products_case(rows, dev):
     """The four square products (receptance, key, value, gate) of `rows` tokens, each over its own blend (width 1600): one
     grouped launch for few tokens, a launch each for many, as the mixer does it."""
@@ -594,6 +670,23 @@ def _grouped_case(which, tokens, dev):
             K.gather_rows(x, rt)
             K.combine_rows(y, pr, stream, TOP, 1.0 / TOP)
         return run, {"bytes": tokens * TOP * width * (2 + 2 + 4) + tokens * width * 8, "flops": tokens * TOP * width}
+    if which == "plainscore":
+        # the router's logits and the choice, sorting with the rows' weights, gathering; the sum is the post-norm's
+        router = torch.randn(EXPERTS, width, device=dev).mul_(0.05).to(torch.bfloat16)
+        stream, y, norm = torch.zeros(tokens, width, device=dev), torch.zeros(rows.shape[0], width, device=dev), torch.ones(width, device=dev)
+
+        def run(i):
+            chosen, weight, _ = K.route_by_score(x, router, EXPERTS, TOP)
+            pr, rt, tg, rw = K.route_by_table(None, chosen, EXPERTS, tile, pair_weight=weight.view(-1))
+            K.gather_rows(x, rt)
+            K.post_norm(stream, y, norm, 1e-6, 0.7, pair_row=pr, rounded_dtype=torch.bfloat16)
+        return run, {"bytes": tokens * TOP * width * (2 + 2 + 4) + tokens * width * 12, "flops": tokens * (TOP + 2 * EXPERTS) * width}
+    if which == "upplain":
+        copies = max(2, min(8, (300 << 20) // (EXPERTS * INNER * width * 2)))
+        weights = [torch.randn(EXPERTS, INNER, width, device=dev).mul_(0.02).to(torch.bfloat16) for _ in range(copies)]
+        scale = torch.rand(rows.shape[0], device=dev)
+        run = lambda i: K.gemm_grouped_tcgen05(rows, weights[i % copies], tile_group, tile, activation="relu2", row_scale=scale)
+        return run, {"bytes": used * INNER * width * 2, "flops": 2 * tokens * TOP * INNER * width}
     if which in ("up", "upsilu"):
         copies = max(2, min(8, (300 << 20) // (EXPERTS * 2 * INNER * width * 2)))
         weights = [torch.randn(EXPERTS, 2 * INNER, width, device=dev).mul_(0.02).to(torch.bfloat16) for _ in range(copies)]
@@ -656,6 +749,10 @@ def build(name, device="cuda:0"):
     sigmoidgate_m<rows> | pairnorm_m<rows> | embedpairs_m<rows> | unitsink_prefill_p<prompts>_t<tokens> |
     unitsink_decode_b<batch>_c<context> | tokenmix_m<rows> | normpair_m<rows> | timescan_p<requests>_t<tokens> | timeprep_p.._t.. |
     timefinish_p.._t.. | timestep_p<requests>_t1 | squares_m<rows> | lowrank_m<rows> | latentwin_prefill_p.._t.. |
+    memscan_p<requests>_t<tokens> | memprep_.. | memgates_.. | memfinish_.. | memstep_p.._t1 (gated; memdecayscan_.. and so on: fixed
+    decays, and a norm over all heads; the suffix _k256v512: 8 heads of 256 by 512) | postnorm_m<rows> | postnormpair_m.. |
+    postnormrows_m.. | grouped_<upplain|plainscore>_m.. (plain experts weighted at their input) | padded_prefill_p.._t.. |
+    padded_decode_b.._c.. |
     latentwin_decode_b.._c.. | latentqprep_m<rows> | perheadturn_m<rows> | grouped_softmax_m<tokens>; attention cases take the suffix _masked (a chunked mask and a gate on every head's
     output)"""
     K.library("core"), K.library("tensor")
@@ -686,6 +783,16 @@ def build(name, device="cuda:0"):
     if parts[0] in ("timescan", "timeprep", "timefinish", "timestep") and "_p" in name:
         entries, tokens = name.split("_p")[1].split("_t")
         return _time_mix_case(int(entries), int(tokens), device, parts[0][4:])
+    if parts[0].startswith("mem") and len(parts) >= 3 and parts[1][0] == "p":
+        # mem[decay]<scan|prep|gates|finish|step>_p<requests>_t<tokens>[_k256v512]
+        fixed = parts[0].startswith("memdecay")
+        big = {"dk": 256, "dv": 512, "heads": 8} if parts[-1] == "k256v512" else {}
+        return _memory_case(int(parts[1][1:]), int(parts[2][1:]), device, parts[0][len("memdecay" if fixed else "mem"):], not fixed, **big)
+    if parts[0] in ("postnorm", "postnormpair", "postnormrows"):
+        return _post_norm_case(int(parts[1][1:]), device, parts[0][len("postnorm"):] or "one")
+    if parts[0] == "padded" and parts[1] in ("prefill", "decode"):
+        a, b = name.split("_", 2)[2][1:].replace("_t", " ").replace("_c", " ").split()
+        return _padded_case(int(a), int(b), device, parts[1] == "decode")
     if name.startswith("groupnorm_m"):
         return _group_norm_shift_case(int(name[len("groupnorm_m"):]), device)
     if name.startswith("depthmix_m"):
@@ -726,7 +833,7 @@ def build(name, device="cuda:0"):
         # retention_p<requests>_t<tokens of each>: prompts; _t1: a decode step of that many requests
         entries, tokens = name.split("_p")[1].split("_t")
         return _retention_case(int(entries), int(tokens), device, finish=name.startswith("retfinish"))
-    if parts[0] == "grouped" and len(parts) == 3 and parts[1] in ("up", "upsilu", "down", "route", "score", "softmax") and parts[2][0] == "m":
+    if parts[0] == "grouped" and len(parts) == 3 and parts[1] in ("up", "upsilu", "upplain", "down", "route", "score", "softmax", "plainscore") and parts[2][0] == "m":
         return _grouped_case(parts[1], int(parts[2][1:]), device)
     if parts[0] == "gemm" and len(parts) == 3 and parts[1] in SHAPES and parts[2][0] == "m":
         return _gemm_case(parts[1], int(parts[2][1:]), device)
