@@ -11,7 +11,7 @@
 // The fade travels as such, not as the decay: a decay near one would lose its distance from one to rounding. f + M - M' is
 // formed as (M - M') + f: where the forget path wins, M - M' is exact and what M' lost to rounding comes back in the fade.
 //
-//   dd_memory_gates    fade, take and exp(-M') of a step's tokens; a warp walks an entry and head, 32 tokens at a time: the
+//   dd_memory_gates    fade, take and exp(-M') of a step's tokens; a block walks an entry and head, 128 tokens at a time: the
 //                      transcendental functions side by side, the maximum one token after the other, so the result does not
 //                      depend on how a prompt was cut
 //   dd_memory_prepare  q, take k and v (and the column of ones) as float32 rows, padded to 16-byte pieces
@@ -34,7 +34,7 @@
 namespace cg = cooperative_groups;
 
 namespace {
-__device__ __forceinline__ float mm_silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float mm_silu(float x) { return __fdividef(x, 1.0f + expf(-x)); }
 __device__ __forceinline__ float mm_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 // The log gates of one token from their projections.
@@ -53,82 +53,105 @@ __device__ __forceinline__ MemoryGates mm_gates(float i, float f, float before, 
     return g;
 }
 
-__global__ void __launch_bounds__(32)
+constexpr int MG_TOKENS = 128;
+
+__global__ void __launch_bounds__(MG_TOKENS)
 memory_gates_kernel(const float* __restrict__ z, int z_stride, float cap, const int* __restrict__ entry_start,
                     const int* __restrict__ entry_slot, float* __restrict__ peak, float* __restrict__ fade,
                     float* __restrict__ take, float* __restrict__ floor_out, int H) {
+    __shared__ __align__(16) float2 logs[MG_TOKENS];     // (i, f) of a token
+    __shared__ float maxima[MG_TOKENS + 1];              // M before the first token, then after every one
     dd_launch_dependents();
-    const int h = blockIdx.x, e = blockIdx.y, lane = threadIdx.x;
+    const int h = blockIdx.x, e = blockIdx.y, tid = threadIdx.x;
     const int start = entry_start[e], end = entry_start[e + 1];
     dd_grid_wait();
     float* mine = peak + (size_t)entry_slot[e] * H + h;
     float M = *mine;
-    float zi = 0.f, zf = 0.f;
-    if (start + lane < end) {
-        zi = z[(size_t)(start + lane) * z_stride + h];
-        zf = z[(size_t)(start + lane) * z_stride + H + h];
-    }
-    for (int t0 = start; t0 < end; t0 += 32) {
-        float i, f;
-        mm_log_gates(zi, zf, cap, i, f);
-        if (t0 + 32 + lane < end) {                      // the next 32 are on their way
-            zi = z[(size_t)(t0 + 32 + lane) * z_stride + h];
-            zf = z[(size_t)(t0 + 32 + lane) * z_stride + H + h];
+    for (int t0 = start; t0 < end; t0 += MG_TOKENS) {
+        const int n = min(MG_TOKENS, end - t0);
+        float i = -INFINITY, f = 0.f;                    // (no token: the maximum stays as it is)
+        if (tid < n) {
+            const float* row = z + (size_t)(t0 + tid) * z_stride + h;
+            mm_log_gates(row[0], row[H], cap, i, f);
         }
-        const int n = min(32, end - t0);
-        float before = 0.f, now = 0.f;
-        for (int j = 0; j < n; ++j) {
-            const float next = fmaxf(__fadd_rn(__shfl_sync(0xffffffffu, f, j), M), __shfl_sync(0xffffffffu, i, j));
-            if (lane == j) { before = M; now = next; }
-            M = next;
+        logs[tid] = make_float2(i, f);
+        __syncthreads();
+        if (tid < 32) {
+            // one warp walks the tokens, all lanes alike; eight at a time, so that their loads lie ahead of the chain
+            if (tid == 0) maxima[0] = M;
+            for (int j = 0; j < n; j += 8) {
+                float2 l[8];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) l[u] = logs[j + u];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) {
+                    M = fmaxf(__fadd_rn(l[u].y, M), l[u].x);
+                    if (tid == u) maxima[j + u + 1] = M;
+                }
+            }
         }
-        if (lane < n) {
-            const MemoryGates g = mm_gates(i, f, before, now);
-            const size_t at = (size_t)(t0 + lane) * H + h;
+        __syncthreads();
+        if (tid < n) {
+            const MemoryGates g = mm_gates(i, f, maxima[tid], maxima[tid + 1]);
+            const size_t at = (size_t)(t0 + tid) * H + h;
             fade[at] = g.fade;
             take[at] = g.take;
             floor_out[at] = g.floor;
         }
     }
-    if (lane == 0 && start < end) *mine = M;
+    if (tid == 0 && start < end) *mine = M;
 }
 
-// A warp owns (token, head).
-template <typename T>
+// Four neighbouring elements from c on (those past n as zeros); WIDE: one load.
+template <typename T, bool WIDE>
+__device__ __forceinline__ float4 mm_load4(const T* row, int c, int n) {
+    if (WIDE && c < n) {
+        if (sizeof(T) == 2) {
+            const uint2 u = *reinterpret_cast<const uint2*>(row + c);
+            return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                               __uint_as_float(u.y & 0xffff0000u));
+        }
+        return *reinterpret_cast<const float4*>(row + c);
+    }
+    float4 x;
+    x.x = c < n ? dd_to_f32(row[c]) : 0.f;
+    x.y = c + 1 < n ? dd_to_f32(row[c + 1]) : 0.f;
+    x.z = c + 2 < n ? dd_to_f32(row[c + 2]) : 0.f;
+    x.w = c + 3 < n ? dd_to_f32(row[c + 3]) : 0.f;
+    return x;
+}
+
+// A thread owns four neighbouring elements of a head's q, k or v; the blocks of grid column t share token t.
+template <typename T, bool WIDE>
 __global__ void __launch_bounds__(256)
 memory_prepare_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int stride, float q_scale,
                       int silu, const float* __restrict__ take, float* __restrict__ q_out, float* __restrict__ k_out,
-                      float* __restrict__ v_out, int n_tokens, int H, int dk, int dv, int ones, int qk_row, int v_row) {
+                      float* __restrict__ v_out, int H, int dk, int dv, int ones, int qk_row, int v_row) {
     dd_launch_dependents();
     dd_grid_wait();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const long long item = (long long)blockIdx.x * 8 + warp;
-    if (item >= (long long)n_tokens * H) return;
-    const int t = (int)(item / H), h = (int)(item % H);
-    const T* qr = q + (size_t)t * stride + (size_t)h * dk;
-    const T* kr = k + (size_t)t * stride + (size_t)h * dk;
-    const T* vr = v + (size_t)t * stride + (size_t)h * dv;
-    const float by = take ? take[item] : 1.0f;
-    auto act = [&](T x) {
-        const float f = dd_to_f32(x);
-        return silu ? mm_silu(f) : f;
-    };
-    for (int c = lane * 4; c < qk_row; c += 128) {
-        float4 a, b;
-        a.x = c < dk ? act(qr[c]) * q_scale : 0.f;
-        a.y = c + 1 < dk ? act(qr[c + 1]) * q_scale : 0.f;
-        a.z = c + 2 < dk ? act(qr[c + 2]) * q_scale : 0.f;
-        a.w = c + 3 < dk ? act(qr[c + 3]) * q_scale : 0.f;
-        b.x = c < dk ? act(kr[c]) * by : 0.f;
-        b.y = c + 1 < dk ? act(kr[c + 1]) * by : 0.f;
-        b.z = c + 2 < dk ? act(kr[c + 2]) * by : 0.f;
-        b.w = c + 3 < dk ? act(kr[c + 3]) * by : 0.f;
-        *reinterpret_cast<float4*>(q_out + (size_t)item * qk_row + c) = a;
-        *reinterpret_cast<float4*>(k_out + (size_t)item * qk_row + c) = b;
+    const int t = blockIdx.x, qk4 = qk_row / 4, v4 = v_row / 4;
+    int piece = blockIdx.y * 256 + threadIdx.x;
+    const int kind = piece < H * qk4 ? 0 : (piece < 2 * H * qk4 ? 1 : 2);
+    piece -= kind * H * qk4;
+    const int per = kind < 2 ? qk4 : v4, h = piece / per, c = (piece - h * per) * 4;
+    if (h >= H) return;
+    const size_t item = (size_t)t * H + h;
+    float4 x;
+    if (kind < 2) x = mm_load4<T, WIDE>((kind ? k : q) + (size_t)t * stride + (size_t)h * dk, c, dk);
+    else x = mm_load4<T, WIDE>(v + (size_t)t * stride + (size_t)h * dv, c, dv);
+    if (silu) { x.x = mm_silu(x.x); x.y = mm_silu(x.y); x.z = mm_silu(x.z); x.w = mm_silu(x.w); }
+    if (kind < 2) {
+        const float by = kind == 0 ? q_scale : (take ? take[item] : 1.0f);
+        *reinterpret_cast<float4*>((kind ? k_out : q_out) + item * qk_row + c) = make_float4(x.x * by, x.y * by, x.z * by, x.w * by);
+        return;
     }
-    auto value = [&](int c) { return c < dv ? act(vr[c]) : (ones && c == dv ? 1.0f : 0.f); };
-    for (int c = lane * 4; c < v_row; c += 128)
-        *reinterpret_cast<float4*>(v_out + (size_t)item * v_row + c) = make_float4(value(c), value(c + 1), value(c + 2), value(c + 3));
+    if (ones && dv - c >= 0 && dv - c < 4) {             // the column of ones
+        if (dv == c) x.x = 1.0f;
+        else if (dv == c + 1) x.y = 1.0f;
+        else if (dv == c + 2) x.z = 1.0f;
+        else x.w = 1.0f;
+    }
+    *reinterpret_cast<float4*>(v_out + item * v_row + c) = x;
 }
 
 __device__ __forceinline__ void mm_copy16(float* dst, const float* src) {
@@ -141,6 +164,29 @@ __device__ __forceinline__ void mm_copy4(float* dst, const float* src) {
 // One row of one column: the update every kernel here uses, rounding by rounding.
 __device__ __forceinline__ float mm_update(float s, float fade, float k, float v) {
     return __fmaf_rn(k, v, __fmaf_rn(-fade, s, s));
+}
+
+// Two neighbouring rows at a time: each half is rounded as the single instruction would round it.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 mm_pack(float lo, float hi) {
+    f32x2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float mm_half_sum(f32x2 x) {
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(x));
+    return __fadd_rn(lo, hi);
+}
+__device__ __forceinline__ f32x2 mm_fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mm_mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
 }
 
 // N sums, of which every one of a column's LPC lanes holds a part: at every exchange (O = 1, 2, 4, .. lanes apart) a lane gives
@@ -219,14 +265,14 @@ memory_scan_kernel(const ScanArgs a) {
     dd_grid_wait();
     const float fixed = a.fade ? 0.f : a.fixed[h];
     float* sp = a.state + ((size_t)a.entry_slot[e] * H + h) * a.cols * DKP + sub * 4;
-    float s[C][R];
+    f32x2 s[C][R / 2];
 #pragma unroll
     for (int c = 0; c < C; ++c) {
         const int col = min(col0 + my_col + c, a.cols - 1);
 #pragma unroll
         for (int p = 0; p < P; ++p) {
-            const float4 x = *reinterpret_cast<const float4*>(sp + (size_t)col * DKP + p * 4 * LPC);
-            s[c][4 * p] = x.x; s[c][4 * p + 1] = x.y; s[c][4 * p + 2] = x.z; s[c][4 * p + 3] = x.w;
+            const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(sp + (size_t)col * DKP + p * 4 * LPC);
+            s[c][2 * p] = x.x; s[c][2 * p + 1] = x.y;
         }
     }
     __syncthreads();                                    // the zeros are written before any copy lands
@@ -254,19 +300,21 @@ memory_scan_kernel(const ScanArgs a) {
         const float* sv = staged + buf * BUF + 2 * MM_TOKENS * DKP + my_col;
         const float* sf = staged + buf * BUF + MM_TOKENS * (2 * DKP + COLS);
         // A token's operands are requested while the token before is worked through.
-        float ops[2][2][R], vv[2][C], ff[2];
+        f32x2 ops[2][2][R / 2], ff[2];
+        float vv[2][C];
         auto fetch = [&](int tt, int slot) {
 #pragma unroll
             for (int w = 0; w < 2; ++w)
 #pragma unroll
                 for (int p = 0; p < P; ++p) {
-                    const float4 x = *reinterpret_cast<const float4*>(sq + (w * MM_TOKENS + tt) * DKP + p * 4 * LPC);
-                    ops[slot][w][4 * p] = x.x; ops[slot][w][4 * p + 1] = x.y; ops[slot][w][4 * p + 2] = x.z; ops[slot][w][4 * p + 3] = x.w;
+                    const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(sq + (w * MM_TOKENS + tt) * DKP + p * 4 * LPC);
+                    ops[slot][w][2 * p] = x.x; ops[slot][w][2 * p + 1] = x.y;
                 }
 #pragma unroll
             for (int c = 0; c < C; ++c) vv[slot][c] = sv[tt * COLS + c];
             // a fixed fade does not touch the tokens past the end either: the state would fade
-            ff[slot] = a.fade ? sf[tt] : (tt < n ? fixed : 0.f);
+            const float lost = -(a.fade ? sf[tt] : (tt < n ? fixed : 0.f));
+            ff[slot] = mm_pack(lost, lost);
         };
         fetch(0, 0);
         // (all sixteen, tokens of zeros among them: one group's exchanges then lie under the next group's products)
@@ -279,18 +327,14 @@ memory_scan_kernel(const ScanArgs a) {
                 fetch(min(tt0 + j + 1, MM_TOKENS - 1), slot ^ 1);
 #pragma unroll
                 for (int c = 0; c < C; ++c) {
+                    const f32x2 value = mm_pack(vv[slot][c], vv[slot][c]);
+                    f32x2 part;
 #pragma unroll
-                    for (int i = 0; i < R; ++i) s[c][i] = mm_update(s[c][i], ff[slot], ops[slot][1][i], vv[slot][c]);
-                    float part[P];
-#pragma unroll
-                    for (int p = 0; p < P; ++p) {
-                        part[p] = 0.f;
-#pragma unroll
-                        for (int i = 4 * p; i < 4 * p + 4; ++i) part[p] = __fmaf_rn(s[c][i], ops[slot][0][i], part[p]);
+                    for (int i = 0; i < R / 2; ++i) {
+                        s[c][i] = mm_fma2(ops[slot][1][i], value, mm_fma2(ff[slot], s[c][i], s[c][i]));
+                        part = i ? mm_fma2(s[c][i], ops[slot][0][i], part) : mm_mul2(s[c][i], ops[slot][0][i]);
                     }
-                    read[j * C + c] = part[0];
-#pragma unroll
-                    for (int p = 1; p < P; ++p) read[j * C + c] = __fadd_rn(read[j * C + c], part[p]);
+                    read[j * C + c] = mm_half_sum(part);
                 }
             }
             const int first = mm_spread_sums<4 * C, 1, LPC>(read, sub);
@@ -313,7 +357,7 @@ memory_scan_kernel(const ScanArgs a) {
             if (col >= a.cols) continue;
 #pragma unroll
             for (int p = 0; p < P; ++p)
-                *reinterpret_cast<float4*>(sp + (size_t)col * DKP + p * 4 * LPC) = make_float4(s[c][4 * p], s[c][4 * p + 1], s[c][4 * p + 2], s[c][4 * p + 3]);
+                *reinterpret_cast<ulonglong2*>(sp + (size_t)col * DKP + p * 4 * LPC) = make_ulonglong2(s[c][2 * p], s[c][2 * p + 1]);
         }
     }
 }
@@ -338,7 +382,7 @@ struct StepArgs {
 };
 
 // Single tokens: token t is entry t. A cluster owns (entry, head), its blocks share the columns out. Gated: every block works
-// the column of n out for itself (it needs n . q); the first block writes it and the maximum, once all have read them.
+// n out for itself (it needs n . q), an element a thread; the first block writes it and the maximum, once all have read them.
 constexpr int ST_THREADS = 256, ST_AHEAD = 2;
 template <typename T, int LPC, bool FUSED>
 __global__ void __launch_bounds__(ST_THREADS)
@@ -346,7 +390,7 @@ memory_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __
                    T* __restrict__ out, const StepArgs a) {
     constexpr int DKP = 8 * LPC, COLS = ST_THREADS / LPC;
     extern __shared__ __align__(16) float sh[];          // q, k [DKP] each, then v and o of the block's columns
-    __shared__ float scratch[8], parts[8];
+    __shared__ float scratch[8], n_parts[8], parts[8];
     dd_launch_dependents();
     const int slice = blockIdx.x, slices = gridDim.x, h = blockIdx.y, e = blockIdx.z;
     cg::cluster_group cluster = cg::this_cluster();
@@ -354,12 +398,12 @@ memory_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int my_col = tid / LPC, sub = tid % LPC;
     const bool gated = a.z != nullptr;
-    const int extra = gated ? 1 : 0;                     // local column 0 is n
     const int per = (a.dv + slices - 1) / slices;
-    const int c_from = min(slice * per, a.dv), mine = min(per, a.dv - c_from), n_cols = mine + extra;
-    float *sq = sh, *sk = sq + DKP, *sv = sk + DKP, *so = sv + per + extra;
+    const int c_from = min(slice * per, a.dv), mine = min(per, a.dv - c_from);
+    float *sq = sh, *sk = sq + DKP, *sv = sk + DKP, *so = sv + per;
     const int slot = a.entry_slot[e];
-    float* base = a.state + ((size_t)slot * a.H + h) * (a.dv + extra) * DKP;
+    float* base = a.state + ((size_t)slot * a.H + h) * (a.dv + (gated ? 1 : 0)) * DKP;
+    float* n_at = base + (size_t)a.dv * DKP + tid;       // (gated, tid < DKP)
     for (int c = tid; c < mine * DKP / 32; c += ST_THREADS)      // the block's columns on their way into L2 (one line a thread)
         asm volatile("prefetch.global.L2 [%0];" ::"l"(base + (size_t)c_from * DKP + (size_t)c * 32));
     dd_grid_wait();
@@ -383,27 +427,32 @@ memory_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __
         sq[i] = i < a.dk ? act(q[row + (size_t)h * a.dk + i]) * a.q_scale : 0.f;
         sk[i] = i < a.dk ? act(k[row + (size_t)h * a.dk + i]) * g.take : 0.f;
     }
-    for (int i = tid; i < n_cols; i += ST_THREADS) sv[i] = i < extra ? 1.0f : act(v[row + (size_t)h * a.dv + c_from + i - extra]);
+    for (int i = tid; i < mine; i += ST_THREADS) sv[i] = act(v[row + (size_t)h * a.dv + c_from + i]);
+    const float n_before = gated && tid < DKP ? *n_at : 0.f;
     __syncthreads();
-    float held[8];                                       // the updated n, of the lanes of local column 0
+    float n_now = 0.f;
+    if (gated) {
+        if (tid < DKP) n_now = mm_update(n_before, g.fade, sk[tid], 1.0f);
+        const float part = dd_warp_sum(tid < DKP ? n_now * sq[tid] : 0.f);
+        if (lane == 0) n_parts[warp] = part;
+    }
     const float4 qa = *reinterpret_cast<const float4*>(sq + sub * 8), qb = *reinterpret_cast<const float4*>(sq + sub * 8 + 4);
     const float4 ka = *reinterpret_cast<const float4*>(sk + sub * 8), kb = *reinterpret_cast<const float4*>(sk + sub * 8 + 4);
     const float qq[8] = {qa.x, qa.y, qa.z, qa.w, qb.x, qb.y, qb.z, qb.w};
     const float kk[8] = {ka.x, ka.y, ka.z, ka.w, kb.x, kb.y, kb.z, kb.w};
-    // where a local column lies in the state
-    auto column = [&](int local) { return base + (size_t)(local < extra ? a.dv : c_from + local - extra) * DKP + sub * 8; };
-    for (int c0 = my_col; c0 - my_col < n_cols; c0 += ST_AHEAD * COLS) {
+    base += (size_t)c_from * DKP + sub * 8;
+    for (int c0 = my_col; c0 - my_col < mine; c0 += ST_AHEAD * COLS) {
         float s[ST_AHEAD][8];
 #pragma unroll
         for (int w = 0; w < ST_AHEAD; ++w) {
-            const float* sp = column(min(c0 + w * COLS, n_cols - 1));
+            const float* sp = base + (size_t)min(c0 + w * COLS, mine - 1) * DKP;
             const float4 x = *reinterpret_cast<const float4*>(sp), y = *reinterpret_cast<const float4*>(sp + 4);
             s[w][0] = x.x; s[w][1] = x.y; s[w][2] = x.z; s[w][3] = x.w; s[w][4] = y.x; s[w][5] = y.y; s[w][6] = y.z; s[w][7] = y.w;
         }
 #pragma unroll
         for (int w = 0; w < ST_AHEAD; ++w) {
             const int c = c0 + w * COLS;
-            const float vv = sv[min(c, n_cols - 1)];
+            const float vv = sv[min(c, mine - 1)];
             float even = 0.f, odd = 0.f;
 #pragma unroll
             for (int i = 0; i < 8; i += 2) {
@@ -415,24 +464,24 @@ memory_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __
             float read = even + odd;
 #pragma unroll
             for (int o = LPC / 2; o > 0; o >>= 1) read += __shfl_xor_sync(0xffffffffu, read, o);
-            if (c < n_cols) {
-                if (c < extra) {
-#pragma unroll
-                    for (int i = 0; i < 8; ++i) held[i] = s[w][i];
-                } else {
-                    float* sp = column(c);
-                    *reinterpret_cast<float4*>(sp) = make_float4(s[w][0], s[w][1], s[w][2], s[w][3]);
-                    *reinterpret_cast<float4*>(sp + 4) = make_float4(s[w][4], s[w][5], s[w][6], s[w][7]);
-                }
+            if (c < mine) {
+                float* sp = base + (size_t)c * DKP;
+                *reinterpret_cast<float4*>(sp) = make_float4(s[w][0], s[w][1], s[w][2], s[w][3]);
+                *reinterpret_cast<float4*>(sp + 4) = make_float4(s[w][4], s[w][5], s[w][6], s[w][7]);
                 if (sub == 0) so[c] = read;
             }
         }
     }
     __syncthreads();
+    float n_dot_q = 0.f;
+    if (gated) {
+#pragma unroll
+        for (int w = 0; w < ST_THREADS / 32; ++w) n_dot_q += n_parts[w];
+    }
     if (FUSED) {
-        const float over = gated ? 1.0f / (fmaxf(fabsf(so[0]), g.floor) + a.den_eps) : 1.0f;
+        const float over = gated ? 1.0f / (fmaxf(fabsf(n_dot_q), g.floor) + a.den_eps) : 1.0f;
         float sum = 0.f;
-        for (int i = extra + tid; i < n_cols; i += ST_THREADS) {
+        for (int i = tid; i < mine; i += ST_THREADS) {
             const float x = so[i] * over;
             so[i] = x;
             sum = fmaf(x, x, sum);
@@ -454,22 +503,18 @@ memory_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __
         const size_t at = (size_t)h * a.dv + c_from;
         for (int i = tid; i < mine; i += ST_THREADS)
             out[(size_t)e * a.out_stride + at + i] =
-                dd_from_f32<T>(so[extra + i] * inv * a.weight[at + i] * mm_sigmoid(dd_to_f32(gate[row + at + i])));
+                dd_from_f32<T>(so[i] * inv * a.weight[at + i] * mm_sigmoid(dd_to_f32(gate[row + at + i])));
     } else {
         float* o = a.o + ((size_t)e * a.H + h) * a.v_row;
-        for (int i = tid; i < mine; i += ST_THREADS) o[c_from + i] = so[extra + i];
+        for (int i = tid; i < mine; i += ST_THREADS) o[c_from + i] = so[i];
         if (gated && slice == 0 && tid == 0) {
-            o[a.dv] = so[0];
+            o[a.dv] = n_dot_q;
             a.floor_out[(size_t)e * a.H + h] = g.floor;
         }
         if (gated && slices > 1) cluster.sync();
     }
     if (gated && slice == 0) {                           // every block of the cluster has read the old n and the old maximum
-        if (my_col == 0) {
-            float* sp = column(0);
-            *reinterpret_cast<float4*>(sp) = make_float4(held[0], held[1], held[2], held[3]);
-            *reinterpret_cast<float4*>(sp + 4) = make_float4(held[4], held[5], held[6], held[7]);
-        }
+        if (tid < DKP) *n_at = n_now;
         if (tid == 0) a.peak[(size_t)slot * a.H + h] = now;
     }
 }
@@ -483,24 +528,28 @@ struct FinishArgs {
     int heads;                   // heads that are normed together: 1 or H
 };
 
-// A team of TEAM threads owns a stretch (a token's head, or a token's heads together); V elements a load.
-template <typename T, int TEAM, int V>
+// A team of TEAM threads owns a stretch (a token's head, or a token's heads together); V elements a load, KEEP loads a thread
+// kept in registers (beyond, it reads again).
+template <typename T, int TEAM, int V, int KEEP>
 __global__ void __launch_bounds__(256)
 memory_finish_kernel(const T* __restrict__ gate, T* __restrict__ out, const FinishArgs a) {
-    constexpr int KEEP = 16 / V;                         // loads a thread keeps in registers; beyond, it reads again
     __shared__ float scratch[8];
     dd_launch_dependents();
     dd_grid_wait();
     const int sub = threadIdx.x % TEAM, per_token = a.H / a.heads;
     const long long stretch = (long long)blockIdx.x * (256 / TEAM) + threadIdx.x / TEAM;
-    if (TEAM == 32 && stretch >= (long long)a.n_tokens * per_token) return;
-    const int t = (int)(stretch / per_token), h0 = (int)(stretch % per_token) * a.heads, size = a.heads * a.dv;
+    const bool none = stretch >= (long long)a.n_tokens * per_token;      // (a team past the end: it still takes part in its warp's sums)
+    const int t = none ? 0 : (int)(stretch / per_token), h0 = none ? 0 : (int)(stretch % per_token) * a.heads;
+    const int size = none ? 0 : a.heads * a.dv;
     const float* row = a.o + (size_t)t * a.H * a.v_row;
+    auto over_of = [&](int h) {
+        return a.floor ? 1.0f / (fmaxf(fabsf(row[(size_t)h * a.v_row + a.dv]), a.floor[(size_t)t * a.H + h]) + a.den_eps) : 1.0f;
+    };
+    const float alone = a.heads == 1 ? over_of(h0) : 1.0f;
     auto load = [&](int c, float* x) {
-        const int h = h0 + c / a.dv;
-        const float* at = row + (size_t)h * a.v_row;
-        const float over = a.floor ? 1.0f / (fmaxf(fabsf(at[a.dv]), a.floor[(size_t)t * a.H + h]) + a.den_eps) : 1.0f;
-        at += c % a.dv;
+        const int h = a.heads == 1 ? h0 : h0 + c / a.dv;
+        const float over = a.heads == 1 ? alone : over_of(h);
+        const float* at = row + (size_t)h * a.v_row + (c - (h - h0) * a.dv);
         if (V == 4) {
             const float4 y = *reinterpret_cast<const float4*>(at);
             x[0] = y.x * over; x[1] = y.y * over; x[2] = y.z * over; x[3] = y.w * over;
@@ -525,7 +574,8 @@ memory_finish_kernel(const T* __restrict__ gate, T* __restrict__ out, const Fini
 #pragma unroll
         for (int i = 0; i < V; ++i) sum = fmaf(x[i], x[i], sum);
     }
-    sum = dd_warp_sum(sum);
+#pragma unroll
+    for (int o = (TEAM < 32 ? TEAM : 32) / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
     if (TEAM > 32) {
         if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = sum;
         __syncthreads();
@@ -569,8 +619,8 @@ int memory_lanes(int dk) {
 template <typename T, int L, bool FUSED>
 int launch_memory_step(const void* q, const void* k, const void* v, const void* gate, void* out, const StepArgs& a, int n_entries,
                        int slices, cudaStream_t s) {
-    const int extra = a.z ? 1 : 0, per = (a.dv + slices - 1) / slices;
-    const size_t smem = (size_t)(2 * 8 * L + 2 * (per + extra)) * sizeof(float);
+    const int per = (a.dv + slices - 1) / slices;
+    const size_t smem = (size_t)(2 * 8 * L + 2 * per) * sizeof(float);
     cudaLaunchConfig_t config = {};
     config.gridDim = dim3(slices, a.H, n_entries);
     config.blockDim = dim3(ST_THREADS);
@@ -601,10 +651,10 @@ int launch_memory_step_sized(int lpc, const void* q, const void* k, const void* 
     }
 }
 
-template <typename T, int TEAM, int V>
+template <typename T, int TEAM, int V, int KEEP>
 int launch_memory_finish(const void* gate, void* out, const FinishArgs& a, cudaStream_t s) {
     const long long stretches = (long long)a.n_tokens * (a.H / a.heads);
-    dd_launch(memory_finish_kernel<T, TEAM, V>, dim3(dd_ceil_div(stretches, 256 / TEAM)), dim3(256), 0, s, (const T*)gate, (T*)out, a);
+    dd_launch(memory_finish_kernel<T, TEAM, V, KEEP>, dim3(dd_ceil_div(stretches, 256 / TEAM)), dim3(256), 0, s, (const T*)gate, (T*)out, a);
     return dd_check_launch("dd_memory_finish");
 }
 
@@ -612,9 +662,13 @@ template <typename T>
 int launch_memory_finish_sized(const void* gate, void* out, const FinishArgs& a, cudaStream_t s) {
     const bool wide = a.dv % 4 == 0 && a.gate_stride % 4 == 0 && a.out_stride % 4 == 0 &&
                       !(((uintptr_t)gate | (uintptr_t)out) & (4 * sizeof(T) - 1)) && !((uintptr_t)a.o & 15);
-    if (a.heads * a.dv <= 512)
-        return wide ? launch_memory_finish<T, 32, 4>(gate, out, a, s) : launch_memory_finish<T, 32, 1>(gate, out, a, s);
-    return wide ? launch_memory_finish<T, 256, 4>(gate, out, a, s) : launch_memory_finish<T, 256, 1>(gate, out, a, s);
+    const int size = a.heads * a.dv;
+    if (!wide) return size <= 512 ? launch_memory_finish<T, 32, 1, 16>(gate, out, a, s) : launch_memory_finish<T, 256, 1, 16>(gate, out, a, s);
+    if (size <= 64) return launch_memory_finish<T, 16, 4, 1>(gate, out, a, s);
+    if (size <= 128) return launch_memory_finish<T, 32, 4, 1>(gate, out, a, s);
+    if (size <= 512) return launch_memory_finish<T, 32, 4, 4>(gate, out, a, s);
+    if (size <= 2048) return launch_memory_finish<T, 256, 4, 2>(gate, out, a, s);
+    return launch_memory_finish<T, 256, 4, 4>(gate, out, a, s);
 }
 }  // namespace
 
@@ -624,7 +678,7 @@ DD_API int dd_memory_gates(const float* z, int z_stride, float cap, const int* e
                            float* peak, float* fade, float* take, float* floor_out, int H, void* stream) {
     if (n_entries <= 0) return 0;
     if (H <= 0 || n_entries > 65535 || !(cap > 0.f) || z_stride < 2 * H) return dd_fail("dd_memory_gates: bad sizes (%d heads)", H);
-    dd_launch(memory_gates_kernel, dim3(H, n_entries), dim3(32), 0, (cudaStream_t)stream, z, z_stride, cap, entry_start, entry_slot,
+    dd_launch(memory_gates_kernel, dim3(H, n_entries), dim3(MG_TOKENS), 0, (cudaStream_t)stream, z, z_stride, cap, entry_start, entry_slot,
               peak, fade, take, floor_out, H);
     return dd_check_launch("dd_memory_gates");
 }
@@ -637,15 +691,17 @@ DD_API int dd_memory_prepare(const void* q, const void* k, const void* v, int st
     if (H <= 0 || dk <= 0 || dv <= 0 || (ones != 0 && ones != 1)) return dd_fail("dd_memory_prepare: bad sizes");
     if (((uintptr_t)q_out | (uintptr_t)k_out | (uintptr_t)v_out) & 15) return dd_fail("dd_memory_prepare: outputs must be 16-byte aligned");
     cudaStream_t s = (cudaStream_t)stream;
-    const int grid = dd_ceil_div((long long)n * H, 8), qk_row = (dk + 3) / 4 * 4, v_row = (dv + ones + 3) / 4 * 4;
-    if (dtype == DD_F32)
-        dd_launch(memory_prepare_kernel<float>, dim3(grid), dim3(256), 0, s, (const float*)q, (const float*)k, (const float*)v, stride,
-                  q_scale, silu, take, q_out, k_out, v_out, n, H, dk, dv, ones, qk_row, v_row);
-    else if (dtype == DD_BF16)
-        dd_launch(memory_prepare_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, s, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k,
-                  (const __nv_bfloat16*)v, stride, q_scale, silu, take, q_out, k_out, v_out, n, H, dk, dv, ones, qk_row, v_row);
-    else
-        return dd_fail("dd_memory_prepare: unknown dtype %d", dtype);
+    const int qk_row = (dk + 3) / 4 * 4, v_row = (dv + ones + 3) / 4 * 4;
+    const int size = dtype == DD_F32 ? 4 : 2;
+    const bool wide = dk % 4 == 0 && dv % 4 == 0 && stride % 4 == 0 && !(((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & (4 * size - 1));
+    const dim3 grid(n, dd_ceil_div((long long)H * (2 * qk_row + v_row) / 4, 256));
+#define DD_PREP(T, WIDE)                                                                                                           \
+    dd_launch(memory_prepare_kernel<T, WIDE>, grid, dim3(256), 0, s, (const T*)q, (const T*)k, (const T*)v, stride, q_scale, silu, take, \
+              q_out, k_out, v_out, H, dk, dv, ones, qk_row, v_row)
+    if (dtype == DD_F32) { if (wide) DD_PREP(float, true); else DD_PREP(float, false); }
+    else if (dtype == DD_BF16) { if (wide) DD_PREP(__nv_bfloat16, true); else DD_PREP(__nv_bfloat16, false); }
+    else return dd_fail("dd_memory_prepare: unknown dtype %d", dtype);
+#undef DD_PREP
     return dd_check_launch("dd_memory_prepare");
 }
 
@@ -662,22 +718,22 @@ DD_API int dd_memory_scan(const float* q, const float* k, const float* v, const 
     a.q = q; a.k = k; a.v = v; a.fade = fade; a.fixed = fixed; a.entry_start = entry_start; a.entry_slot = entry_slot;
     a.state = state; a.out = out; a.H = H; a.cols = dv + ones; a.qk_row = (dk + 3) / 4 * 4; a.v_row = (dv + ones + 3) / 4 * 4;
     cudaStream_t s = (cudaStream_t)stream;
-    // blocks of 16 columns (more where a warp holds more)
-#define DD_SCAN(R, C, L)                                                                                                \
+    // blocks of CB columns (more where a warp holds more)
+#define DD_SCAN(R, C, L, CB)                                                                                            \
     do {                                                                                                                \
-        constexpr int TH = L * 16 / C > 32 ? L * 16 / C : 32, COLS = TH / L * C;                                        \
+        constexpr int TH = L * CB / C > 32 ? L * CB / C : 32, COLS = TH / L * C;                                        \
         const size_t smem = (size_t)2 * (MM_TOKENS * (2 * R * L + COLS + 1)) * sizeof(float);                           \
         if (smem > 48 * 1024)                                                                                           \
             cudaFuncSetAttribute(memory_scan_kernel<R, C, L, TH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         dd_launch_in_order(memory_scan_kernel<R, C, L, TH>, dim3(dd_ceil_div(a.cols, COLS), H, n_entries), dim3(TH), smem, s, a);     \
     } while (0)
     switch (8 * memory_lanes(dk)) {
-        case 8: DD_SCAN(4, 4, 2); break;
-        case 16: DD_SCAN(4, 4, 4); break;
-        case 32: DD_SCAN(4, 4, 8); break;
-        case 64: DD_SCAN(4, 4, 16); break;
-        case 128: DD_SCAN(4, 4, 32); break;
-        default: DD_SCAN(8, 2, 32); break;
+        case 8: DD_SCAN(4, 4, 2, 16); break;
+        case 16: DD_SCAN(4, 4, 4, 16); break;
+        case 32: DD_SCAN(4, 4, 8, 16); break;
+        case 64: DD_SCAN(8, 2, 8, 16); break;
+        case 128: DD_SCAN(8, 2, 16, 16); break;
+        default: DD_SCAN(8, 4, 32, 32); break;
     }
 #undef DD_SCAN
     return dd_check_launch("dd_memory_scan");

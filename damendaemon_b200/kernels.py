@@ -589,11 +589,13 @@ def memory_scan(q, k, v, fade, entry_start, entry_slot, state, head_dim, value_d
 
 
 def memory_slices(entries, heads, head_dim, value_dim, device):
-    """Into how many blocks ``memory_step`` cuts a head's columns: as many as fill the GPU about twice, while a block keeps at
-    least the columns its threads hold at once."""
-    lanes = memory_state_shape(heads, head_dim, value_dim, False)[2] // 8
+    """Into how many blocks ``memory_step`` cuts a head's columns, while a block keeps at least the columns its threads hold at
+    once (two each): as many as give every SM four blocks, or leave a block no more than 128 KB of state (measured)."""
+    rows = memory_state_shape(heads, head_dim, value_dim, False)[2]
+    at_once = 2 * max(1, 256 * 8 // rows)
     slices = 1
-    while slices < 8 and entries * heads * slices * 2 <= 2 * sm_count(device) and value_dim >= 2 * slices * max(1, 256 // lanes):
+    while slices < 8 and value_dim >= 2 * slices * at_once and \
+            (entries * heads * slices * 2 <= 4 * sm_count(device) or value_dim * rows * 4 > slices * 128 * 1024):
         slices *= 2
     return slices
 
