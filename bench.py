@@ -392,7 +392,7 @@ DOZETAR_KERNEL_PAIRS = [     # (a kernel of Dozetar, the like kernel of the clos
     ("memscan_p2_t1024_k256v512", "timescan_p2_t1024"), ("memstep_p8_t1_k256v512", "timestep_p8_t1"), ("memstep_p64_t1_k256v512", "timestep_p64_t1"),
     ("memdecayprep_p2_t1024", "timeprep_p2_t1024"), ("memdecayscan_p2_t1024", "retention_p2_t1024"), ("memdecayfinish_p2_t1024", "retfinish_p2_t1024"),
     ("memdecaystep_p8_t1", "retention_p8_t1"), ("memdecaystep_p64_t1", "retention_p64_t1"), ("memdecayfinish_p8_t1", "retfinish_p8_t1"),
-    ("widenorm_m2048", "headnorm_m2048"), ("widenorm_m8", "headnorm_m8"),
+    ("widenormpairs_m2048", "headnorm_m2048"), ("widenormpairs_m8", "headnorm_m8"),
     ("sinks_prefill_p2_t1024", "sinks_prefill_p2_t1024"), ("sinks_decode_b8_c768", "sinks_decode_b8_c768"),
     ("padded_prefill_p2_t1024", "sinks_prefill_p2_t1024"), ("padded_decode_b8_c768", "sinks_decoderows_b8_c768"),
     ("padded_decode_b64_c768", "sinks_decoderows_b64_c768"),

@@ -353,15 +353,16 @@ def _tanh_norm_case(rows, dev):
     return run, {"bytes": rows * width * 6, "flops": 10 * rows * width}
 
 
-def _wide_norm_case(rows, dev):
-    """Queries and keys of `rows` tokens (25 + 25 heads of 64) normed over the whole projection and rotated in halves."""
+def _wide_norm_case(rows, dev, interleaved=False):
+    """Queries and keys of `rows` tokens (25 + 25 heads of 64) normed over the whole projection and rotated in halves (or in
+    neighbouring pairs)."""
     copies = max(2, min(24, (300 << 20) // (rows * 3 * H * D * 2)))
     bufs = [torch.randn(rows, 3 * H * D + 32, device=dev).to(torch.bfloat16) for _ in range(copies)]
     pos = torch.arange(rows, dtype=torch.int32, device=dev) % 1024
     freqs = (10000.0 ** (-torch.arange(D // 2, dtype=torch.float64) * 2 / D)).float().to(dev)
     wq, wk = torch.ones(H * D, device=dev), torch.ones(H * D, device=dev)
     run = lambda i: K.wide_norm_rotary(bufs[i % copies][:, :H * D], bufs[i % copies][:, H * D:2 * H * D], pos, wq, wk, 1e-6, H, H, D,
-                                       freqs=freqs, interleaved=False)
+                                       freqs=freqs, interleaved=interleaved)
     return run, {"bytes": rows * 2 * H * D * 4, "flops": 10 * rows * H * D}
 
 
@@ -744,7 +745,7 @@ def build(name, device="cuda:0"):
     retfinish_p<requests>_t<tokens> | groupnorm_m<rows> | depthmix_m<rows> | delta_p<requests>_t<tokens> | deltaprep_p.._t.. |
     deltafinish_p.._t.. | latent_prefill_p<prompts>_t<tokens> | latent_decode_b<batch>_c<context> | latentprep_m<rows> |
     perhead_m<rows> | perheadup_m<rows> | sinks_prefill_p<prompts>_t<tokens> | sinks_decode_b<batch>_c<context> (and
-    sinks_prefillrows_.., sinks_decoderows_..: through the general kernel) | tanhnorm_m<rows> | widenorm_m<rows> |
+    sinks_prefillrows_.., sinks_decoderows_..: through the general kernel) | tanhnorm_m<rows> | widenorm_m<rows> | widenormpairs_m<rows> |
     ssmconv_p<requests>_t<tokens> | ssmscan_p.._t.. | ssmfinish_p.._t.. | rglrugates_p.._t.. | rglruscan_p.._t.. |
     sigmoidgate_m<rows> | pairnorm_m<rows> | embedpairs_m<rows> | unitsink_prefill_p<prompts>_t<tokens> |
     unitsink_decode_b<batch>_c<context> | tokenmix_m<rows> | normpair_m<rows> | timescan_p<requests>_t<tokens> | timeprep_p.._t.. |
@@ -762,6 +763,8 @@ def build(name, device="cuda:0"):
     parts = name.split("_")
     if name.startswith("tanhnorm_m"):
         return _tanh_norm_case(int(name[len("tanhnorm_m"):]), device)
+    if name.startswith("widenormpairs_m"):
+        return _wide_norm_case(int(name[len("widenormpairs_m"):]), device, interleaved=True)
     if name.startswith("widenorm_m"):
         return _wide_norm_case(int(name[len("widenorm_m"):]), device)
     if parts[0] in ("ssmconv", "ssmscan", "ssmfinish", "rglrugates", "rglruscan") and "_p" in name:

@@ -429,6 +429,9 @@ memory_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __
     }
     for (int i = tid; i < mine; i += ST_THREADS) sv[i] = act(v[row + (size_t)h * a.dv + c_from + i]);
     const float n_before = gated && tid < DKP ? *n_at : 0.f;
+    const size_t at = (size_t)h * a.dv + c_from;
+    // the gate and weight of a thread's first element, ready when the sum of squares is
+    const float gate_ahead = FUSED && tid < mine ? dd_to_f32(gate[row + at + tid]) : 0.f, weight_ahead = FUSED && tid < mine ? a.weight[at + tid] : 0.f;
     __syncthreads();
     float n_now = 0.f;
     if (gated) {
@@ -500,10 +503,10 @@ memory_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __
             for (int w = 0; w < slices; ++w) sum += parts[w];
         }
         const float inv = 1.0f / sqrtf(sum / (float)a.dv + a.eps);
-        const size_t at = (size_t)h * a.dv + c_from;
-        for (int i = tid; i < mine; i += ST_THREADS)
-            out[(size_t)e * a.out_stride + at + i] =
-                dd_from_f32<T>(so[i] * inv * a.weight[at + i] * mm_sigmoid(dd_to_f32(gate[row + at + i])));
+        for (int i = tid; i < mine; i += ST_THREADS) {
+            const float z = i == tid ? gate_ahead : dd_to_f32(gate[row + at + i]), w = i == tid ? weight_ahead : a.weight[at + i];
+            out[(size_t)e * a.out_stride + at + i] = dd_from_f32<T>(so[i] * inv * w * mm_sigmoid(z));
+        }
     } else {
         float* o = a.o + ((size_t)e * a.H + h) * a.v_row;
         for (int i = tid; i < mine; i += ST_THREADS) o[c_from + i] = so[i];
@@ -535,12 +538,20 @@ __global__ void __launch_bounds__(256)
 memory_finish_kernel(const T* __restrict__ gate, T* __restrict__ out, const FinishArgs a) {
     __shared__ float scratch[8];
     dd_launch_dependents();
-    dd_grid_wait();
     const int sub = threadIdx.x % TEAM, per_token = a.H / a.heads;
     const long long stretch = (long long)blockIdx.x * (256 / TEAM) + threadIdx.x / TEAM;
     const bool none = stretch >= (long long)a.n_tokens * per_token;      // (a team past the end: it still takes part in its warp's sums)
     const int t = none ? 0 : (int)(stretch / per_token), h0 = none ? 0 : (int)(stretch % per_token) * a.heads;
     const int size = none ? 0 : a.heads * a.dv;
+    const float* w = a.weight + (size_t)h0 * a.dv;
+    float weights[KEEP][V];                              // (parameters: read before the wait for the kernel before)
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int c = (sub + j * TEAM) * V;
+#pragma unroll
+        for (int i = 0; i < V; ++i) weights[j][i] = c < size ? w[c + i] : 0.f;
+    }
+    dd_grid_wait();
     const float* row = a.o + (size_t)t * a.H * a.v_row;
     auto over_of = [&](int h) {
         return a.floor ? 1.0f / (fmaxf(fabsf(row[(size_t)h * a.v_row + a.dv]), a.floor[(size_t)t * a.H + h]) + a.den_eps) : 1.0f;
@@ -557,13 +568,24 @@ memory_finish_kernel(const T* __restrict__ gate, T* __restrict__ out, const Fini
             x[0] = *at * over;
         }
     };
-    float kept[KEEP][V];
+    const T* g = gate + (size_t)t * a.gate_stride + (size_t)h0 * a.dv;
+    T* dst = out + (size_t)t * a.out_stride + (size_t)h0 * a.dv;
+    auto gate_of = [&](int c, float* z) {
+        __align__(16) T gv[V];
+        if (V == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(gv) = *reinterpret_cast<const uint2*>(g + c);
+        else if (V == 4) *reinterpret_cast<uint4*>(gv) = *reinterpret_cast<const uint4*>(g + c);
+        else gv[0] = g[c];
+#pragma unroll
+        for (int i = 0; i < V; ++i) z[i] = dd_to_f32(gv[i]);
+    };
+    float kept[KEEP][V], gates[KEEP][V];
     float sum = 0.f;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
         const int c = (sub + j * TEAM) * V;
         if (c < size) {
             load(c, kept[j]);
+            gate_of(c, gates[j]);                        // (ready when the sum is)
 #pragma unroll
             for (int i = 0; i < V; ++i) sum = fmaf(kept[j][i], kept[j][i], sum);
         }
@@ -584,16 +606,10 @@ memory_finish_kernel(const T* __restrict__ gate, T* __restrict__ out, const Fini
         for (int w = 0; w < 8; ++w) sum += scratch[w];
     }
     const float inv = 1.0f / sqrtf(sum / (float)size + a.eps);
-    const T* g = gate + (size_t)t * a.gate_stride + (size_t)h0 * a.dv;
-    const float* w = a.weight + (size_t)h0 * a.dv;
-    T* dst = out + (size_t)t * a.out_stride + (size_t)h0 * a.dv;
-    auto store = [&](int c, const float* x) {
-        __align__(16) T gv[V], y[V];
-        if (V == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(gv) = *reinterpret_cast<const uint2*>(g + c);
-        else if (V == 4) *reinterpret_cast<uint4*>(gv) = *reinterpret_cast<const uint4*>(g + c);
-        else gv[0] = g[c];
+    auto store = [&](int c, const float* x, const float* z, const float* by) {
+        __align__(16) T y[V];
 #pragma unroll
-        for (int i = 0; i < V; ++i) y[i] = dd_from_f32<T>(x[i] * inv * w[c + i] * mm_sigmoid(dd_to_f32(gv[i])));
+        for (int i = 0; i < V; ++i) y[i] = dd_from_f32<T>(x[i] * inv * by[i] * mm_sigmoid(z[i]));
         if (V == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(dst + c) = *reinterpret_cast<const uint2*>(y);
         else if (V == 4) *reinterpret_cast<uint4*>(dst + c) = *reinterpret_cast<const uint4*>(y);
         else dst[c] = y[0];
@@ -601,12 +617,13 @@ memory_finish_kernel(const T* __restrict__ gate, T* __restrict__ out, const Fini
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
         const int c = (sub + j * TEAM) * V;
-        if (c < size) store(c, kept[j]);
+        if (c < size) store(c, kept[j], gates[j], weights[j]);
     }
     for (int c = (sub + KEEP * TEAM) * V; c < size; c += TEAM * V) {
-        float x[V];
+        float x[V], z[V];
         load(c, x);
-        store(c, x);
+        gate_of(c, z);
+        store(c, x, z, w + c);
     }
 }
 

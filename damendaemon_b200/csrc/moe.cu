@@ -157,13 +157,18 @@ route_by_score_kernel(const T* __restrict__ y, int ldy, const T* __restrict__ ro
         for (int j = 0; j < ROWS; ++j) acc[j] = 0.f;
         if (wide) {
             for (int c = (warp * 32 + lane) * V; c < width; c += 128 * V) {
+                // (no branch between the rows: all their loads are requested before the first product; sums of rows past the
+                // last are of the last row again, and dropped)
+                uint4 raw[ROWS];
+#pragma unroll
+                for (int j = 0; j < ROWS; ++j)
+                    raw[j] = *reinterpret_cast<const uint4*>(router + (size_t)min(e0 + j, n_rows - 1) * ldr + c);
                 float xv[V];
                 RoutePiece<T>::load(x + c, xv);
 #pragma unroll
                 for (int j = 0; j < ROWS; ++j) {
-                    if (e0 + j >= n_rows) break;
                     float wv[V];
-                    RoutePiece<T>::load(router + (size_t)(e0 + j) * ldr + c, wv);
+                    RoutePiece<T>::load(reinterpret_cast<const T*>(&raw[j]), wv);
 #pragma unroll
                     for (int i = 0; i < V; ++i) acc[j] = fmaf(xv[i], wv[i], acc[j]);
                 }

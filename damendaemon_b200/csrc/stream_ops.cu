@@ -78,6 +78,76 @@ norm_pair_add_kernel(float* __restrict__ x, const float* __restrict__ left, cons
         x[at + c] += half * (left[at + c] * rl * wl[c] + right[at + c] * rr * wr[c]);
 }
 
+// A block owns a token; a thread holds KEEP 16-byte pieces of its row (queries, then keys) in registers from the load that also
+// sums the squares to the store. Pairs are neighbours and lie within a piece. Weights, cosines and sines are ready before the
+// wait for the kernel before.
+template <typename T, int KEEP>
+__global__ void __launch_bounds__(256)
+wide_norm_pieces_kernel(T* __restrict__ q, T* __restrict__ k, int stride, const int* __restrict__ positions,
+                        const float* __restrict__ freqs, const float* __restrict__ qw, const float* __restrict__ kw, float eps,
+                        int nq, int nk, int d, int n_pairs) {
+    constexpr int PIECE = 16 / sizeof(T);
+    extern __shared__ float wn_turns[];                  // cosine and sine of every pair
+    __shared__ float sums[2][8];
+    dd_launch_dependents();
+    const int t = blockIdx.x, threads = blockDim.x;
+    const float position = (float)positions[t];
+    for (int i = threadIdx.x; i < n_pairs; i += threads) sincosf(position * freqs[i], &wn_turns[2 * i + 1], &wn_turns[2 * i]);
+    float w[KEEP][PIECE];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int c = (threadIdx.x + j * threads) * PIECE;
+        const float* from = c < nq ? (qw ? qw + c : nullptr) : (c < nq + nk && kw ? kw + (c - nq) : nullptr);
+#pragma unroll
+        for (int i = 0; i < PIECE; ++i) w[j][i] = from ? from[i] : 1.0f;
+    }
+    dd_grid_wait();
+    T* qr = q + (size_t)t * stride;
+    T* kr = k ? k + (size_t)t * stride : nullptr;
+    float x[KEEP][PIECE];
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int c = (threadIdx.x + j * threads) * PIECE;
+        if (c >= nq + nk) continue;
+        __align__(16) T piece[PIECE];
+        *reinterpret_cast<uint4*>(piece) = *reinterpret_cast<const uint4*>(c < nq ? qr + c : kr + (c - nq));
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < PIECE; ++i) { x[j][i] = dd_to_f32(piece[i]); s = fmaf(x[j][i], x[j][i], s); }
+        if (c < nq) sq += s; else sk += s;
+    }
+    sq = dd_warp_sum(sq);
+    sk = dd_warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) { sums[0][threadIdx.x >> 5] = sq; sums[1][threadIdx.x >> 5] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+    for (int i = 0; i < (threads >> 5); ++i) { sq += sums[0][i]; sk += sums[1][i]; }
+    const float rq = qw ? rsqrtf(sq / (float)nq + eps) : 1.0f;
+    const float rk = (kw && nk) ? rsqrtf(sk / (float)nk + eps) : 1.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int c = (threadIdx.x + j * threads) * PIECE;
+        if (c >= nq + nk) continue;
+        const float r = c < nq ? rq : rk;
+        const int within = (c < nq ? c : c - nq) % d;
+        __align__(16) T piece[PIECE];
+#pragma unroll
+        for (int i = 0; i < PIECE; i += 2) {
+            float u = x[j][i] * r * w[j][i], v = x[j][i + 1] * r * w[j][i + 1];
+            if (within < 2 * n_pairs) {
+                const float2 turn = *reinterpret_cast<const float2*>(&wn_turns[within + i]);
+                const float tu = u * turn.x - v * turn.y;
+                v = v * turn.x + u * turn.y;
+                u = tu;
+            }
+            piece[i] = dd_from_f32<T>(u);
+            piece[i + 1] = dd_from_f32<T>(v);
+        }
+        *reinterpret_cast<uint4*>(c < nq ? qr + c : kr + (c - nq)) = *reinterpret_cast<const uint4*>(piece);
+    }
+}
+
 // A block owns a token. Its cosines and sines are computed once (before the wait for the kernel before: they depend on the
 // position only); the token's queries and keys are brought into shared memory as float32 in one pass of 16-byte loads that
 // also sums their squares; pairs are rotated there, and one pass of 16-byte stores writes the row back. STAGED false: rows
@@ -242,6 +312,20 @@ DD_API int dd_wide_norm_rotary(void* q, void* k, int stride, const int* position
                         (k == nullptr || (uintptr_t)k % 16 == 0) && table + (size_t)(nq + nk) * 4 <= 40 * 1024;
     const size_t smem = table + (staged ? (size_t)(nq + nk) * 4 : 0);
     const int threads = (nq + nk) >= 2048 ? 256 : 128;
+    // neighbouring pairs within 16-byte pieces: the row stays in registers
+    const int pieces = (nq + nk) / piece;
+    if (staged && interleaved && d % piece == 0 && 2 * n_pairs % piece == 0 && pieces <= 4 * 256) {
+        const int block = pieces <= 128 ? 128 : 256, keep = pieces <= 256 ? 1 : (pieces <= 512 ? 2 : 4);
+#define WN_PIECES(T, KEEP) dd_launch(wide_norm_pieces_kernel<T, KEEP>, dim3(n_tokens), dim3(block), 2 * n_pairs * sizeof(float), s, (T*)q, \
+                                     (T*)k, stride, positions, freqs, qw, kw, eps, nq, nk, d, n_pairs)
+#define WN_PIECES_T(T) do { if (keep == 1) WN_PIECES(T, 1); else if (keep == 2) WN_PIECES(T, 2); else WN_PIECES(T, 4); } while (0)
+        if (dtype == DD_F32) WN_PIECES_T(float);
+        else if (dtype == DD_BF16) WN_PIECES_T(__nv_bfloat16);
+        else return dd_fail("dd_wide_norm_rotary: unknown dtype %d", dtype);
+#undef WN_PIECES_T
+#undef WN_PIECES
+        return dd_check_launch("dd_wide_norm_rotary");
+    }
 #define WN_LAUNCH(T, STAGED) dd_launch(wide_norm_rotary_kernel<T, STAGED>, dim3(n_tokens), dim3(threads), smem, s, (T*)q, (T*)k, stride, \
                                        positions, freqs, qw, kw, eps, q_heads, k_heads, d, n_pairs, interleaved)
     if (dtype == DD_F32) { if (staged) WN_LAUNCH(float, true); else WN_LAUNCH(float, false); }
