@@ -516,28 +516,28 @@ def godotar_configs(size, layers, vocab=50257):
 def dozetar_configs(size, layers, vocab=50257):
     """Godotar (layers of time mixing; its looped mix with experts), Zokanex (retention layers; its mix with experts) and Dozetar
     models whose layers have one size: matrix memories alone; parallel layers alone; and memories and parallel layers in turn (a
-    parallel layer as every third); each with experts of Zokanex's sizes in every layer, and the last also with value heads of 48
-    and key heads of 96 (whole tiles padded)."""
+    parallel layer as every third); each with experts of Zokanex's sizes in every layer, and the last also with value heads of 56
+    and key heads of 112 (prompt tiles padded)."""
     z = DESIGN_SIZES[size]
     out = {k: v for k, v in godotar_configs(size, layers, vocab).items() if k in ("godotar_wkv_dense", "godotar_looped_experts")}
     out.update({k: v for k, v in zokanex_configs(size, layers, vocab).items() if k in ("zokanex_retention_dense", "zokanex_mixed_experts")})
     heads = z["heads"]
-    memory = {"heads": heads, "dim": 64, "vdim": 64, "gate_cap": 12.0}
+    memory = {"heads": heads, "dim": 64, "vdim": 64, "gate_cap": 10.0}
     decay = [1.0 - 2.0 ** -(1 + 9 * h / max(1, heads - 1)) for h in range(heads)]
 
     def parallel(dim, vdim):
         left = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "rot": {"dims": dim // 2, "base": 10000.0},
-                "mask": {"size": 1024, "keep_first": 4}}
-        return {"left": left, "right": {"heads": heads, "dim": 64, "vdim": 64, "decay": decay}, "left_scale": 0.6, "right_scale": 0.5}
+                "mask": {"size": 1024, "keep_first": 8}}
+        return {"left": left, "right": {"heads": heads, "dim": 64, "vdim": 64, "decay": decay}, "left_scale": 0.8, "right_scale": 0.4}
     moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["expert_ff"]}}
 
     def model(entries):
-        return {"architecture": "Dozetar", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.7,
-                "logit_softcap": 30.0, "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in entries]}
+        return {"architecture": "Dozetar", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.9,
+                "logit_softcap": 20.0, "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in entries]}
     out["dozetar_memory_experts"] = model([("mlstm", memory)] * layers)
     out["dozetar_parallel_experts"] = model([("parallel", parallel(64, 64))] * layers)
     out["dozetar_mixed_experts"] = model([("parallel", parallel(64, 64)) if i % 3 == 1 else ("mlstm", memory) for i in range(layers)])
-    out["dozetar_mixed_96_48_experts"] = model([("parallel", parallel(96, 48)) if i % 3 == 1 else ("mlstm", memory) for i in range(layers)])
+    out["dozetar_mixed_112_56_experts"] = model([("parallel", parallel(112, 56)) if i % 3 == 1 else ("mlstm", memory) for i in range(layers)])
     return out
 
 

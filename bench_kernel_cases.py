@@ -517,11 +517,11 @@ def _memory_case(entries, length, dev, which, gated=True, dk=D, dv=D, heads=H):
     out = torch.empty(tokens, inner, device=dev, dtype=torch.bfloat16)
     silu = not gated
     if which == "step":
-        more = dict(weight=weight, eps=1e-6, den_eps=1e-6, gates=(z, 12.0, peak), out=out) if gated else dict(fade=fade, silu=True)
+        more = dict(weight=weight, eps=1e-6, den_eps=1e-6, gates=(z, 10.0, peak), out=out) if gated else dict(fade=fade, silu=True)
         run = lambda i: K.memory_step(*split(projs[i % copies]), slot, states[i % copies], heads, dk, dv, **more)
         return run, {"bytes": state_bytes + tokens * 2 * (2 * qk + 3 * inner), "flops": 5 * tokens * heads * shape[1] * dk, "fp32": True}
     if which == "gates":
-        run = lambda i: K.memory_gates(z, 12.0, start, slot, peak)
+        run = lambda i: K.memory_gates(z, 10.0, start, slot, peak)
         return run, {"bytes": tokens * heads * 20, "flops": 40 * tokens * heads, "fp32": True}
     take = torch.ones(tokens, heads, device=dev) if gated else None
     if which == "prep":
@@ -547,20 +547,20 @@ def _post_norm_case(rows, dev, which):
     a, b = ([torch.randn(rows * (2 if which == "rows" else 1), width, device=dev) for _ in range(copies)] for _ in range(2))
     w = torch.ones(width, device=dev)
     pair = torch.randperm(2 * rows, device=dev).to(torch.int32)
-    terms = {"one": lambda i: {}, "pair": lambda i: {"other": b[i], "scale": 0.6, "other_scale": 0.5}, "rows": lambda i: {"pair_row": pair}}[which]
-    run = lambda i: K.post_norm(x[i % copies], a[i % copies], w, 1e-6, 0.7, rounded_dtype=torch.bfloat16, **terms(i % copies))
+    terms = {"one": lambda i: {}, "pair": lambda i: {"other": b[i], "scale": 0.8, "other_scale": 0.4}, "rows": lambda i: {"pair_row": pair}}[which]
+    run = lambda i: K.post_norm(x[i % copies], a[i % copies], w, 1e-6, 0.9, rounded_dtype=torch.bfloat16, **terms(i % copies))
     return run, {"bytes": rows * width * (10 + (4 if which == "one" else 8)), "flops": 6 * rows * width}
 
 
-def _padded_case(batch, length, dev, decode, dk=96, dv=48, heads=H):
-    """Attention whose value heads (48) are smaller than its key heads (96), with a window that holds the whole context, kept first
+def _padded_case(batch, length, dev, decode, dk=112, dv=56, heads=H):
+    """Attention whose value heads (56) are smaller than its key heads (112), with a window that holds the whole context, kept first
     keys and a sink: prompts in padded tiles, single tokens through the general kernel."""
     tokens, n_pages = (batch if decode else batch * length), batch * (-(-length // PAGE))
     copies = max(2, min(12, (300 << 20) // (batch * length * heads * (dk + dv) * 2)))
     caches = [torch.randn(n_pages, heads * PAGE * (dk + dv), device=dev).to(torch.bfloat16) for _ in range(copies)]
     table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(batch, -1)
     q = torch.randn(tokens, heads * dk, device=dev).to(torch.bfloat16)
-    kw = dict(window=1024 * (-(-length // 1024)), keep_first=4, sink=torch.zeros(heads, device=dev), kv_heads=heads, v_dim=dv)
+    kw = dict(window=1024 * (-(-length // 1024)), keep_first=8, sink=torch.zeros(heads, device=dev), kv_heads=heads, v_dim=dv)
     if decode:
         ent = torch.arange(batch, dtype=torch.int32, device=dev)
         pos = torch.full((batch,), length - 1, dtype=torch.int32, device=dev)
@@ -680,7 +680,7 @@ def _grouped_case(which, tokens, dev):
             chosen, weight, _ = K.route_by_score(x, router, EXPERTS, TOP)
             pr, rt, tg, rw = K.route_by_table(None, chosen, EXPERTS, tile, pair_weight=weight.view(-1))
             K.gather_rows(x, rt)
-            K.post_norm(stream, y, norm, 1e-6, 0.7, pair_row=pr, rounded_dtype=torch.bfloat16)
+            K.post_norm(stream, y, norm, 1e-6, 0.9, pair_row=pr, rounded_dtype=torch.bfloat16)
         return run, {"bytes": tokens * TOP * width * (2 + 2 + 4) + tokens * width * 12, "flops": tokens * (TOP + 2 * EXPERTS) * width}
     if which == "upplain":
         copies = max(2, min(8, (300 << 20) // (EXPERTS * INNER * width * 2)))

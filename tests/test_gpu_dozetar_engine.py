@@ -11,7 +11,7 @@ pytestmark = pytest.mark.gpu
 
 LENGTHS = {"A": [1, 5, 19, 20, 21, 41, 100, 130], "B": [2, 6, 7, 8, 15, 50, 64, 90], "C": [1, 99, 100, 101, 134, 260, 300, 201],
            "D": [1, 32, 33, 34, 67, 150, 9, 99], "E": [1, 49, 50, 51, 128, 129, 260, 77]}
-FLOAT32_TOL = 1e-3       # logits reach several tens; a head's read-out that nearly vanishes before its norm amplifies rounding
+FLOAT32_TOL = 2e-4
 TOL = {}
 
 
@@ -25,7 +25,10 @@ def models():
             reference = plain_tensors(tensors)
             want = {r: plain.forward(config, reference, t).float() for r, t in requests.items()}
             out[name, dtype] = (config, tensors, requests, want)
-            TOL[name, dtype] = FLOAT32_TOL
+            # (a head's read-out that nearly vanishes before it is divided by its root mean square amplifies rounding: four times
+            # what float32 does to the plain implementation itself comes on top)
+            TOL[name, dtype] = FLOAT32_TOL + 4.0 * max((plain.forward(config, tensors, t) - want[r]).abs().max().item()
+                                                       for r, t in requests.items()) if dtype == "float32" else None
             if dtype == "bfloat16":
                 # the root mean square of a row's error, against three times what rounding the stored activations to
                 # bfloat16 does to the plain implementation's own rows (a wrong or missing key, or a lost state, moves
@@ -126,7 +129,7 @@ def test_mixed_batches_with_pages_and_slots_used_again(models, name, dtype):
         again = replay(engine, builder)
         for r in requests:
             for p in again[r]:
-                assert (again[r][p] - alone[r][p]).abs().max().item() < FLOAT32_TOL / 2, (r, p)
+                assert (again[r][p] - alone[r][p]).abs().max().item() < TOL[name, dtype] / 2, (r, p)
 
 
 def test_a_windowed_layer_gives_its_pages_back(models):
